@@ -6,6 +6,7 @@ from .taredra import TaredraConfig
 from .disorax import DisoraxConfig
 from .zadunex import ZadunexConfig
 from .fogizen import FogizenConfig
+from .zefapel import ZefapelConfig
 from .registry import (Architecture, architecture_name, get_architecture, known_architectures, preset_config,
                        read_config, register_architecture)
 

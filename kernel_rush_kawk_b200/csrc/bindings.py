@@ -54,18 +54,23 @@ _SIGNATURES = {
 _MIX_SIGNATURES = {
     "krk_embed_scaled": [_P, _P, _P, c_int, c_int, c_int, c_float, _P, c_int, _P, c_int],
     "krk_rmsnorm_wide": [_P, _P, _P, _P, _P, c_float, c_int, c_int, c_float, _P, c_float, _P, _P, c_int, _P],
+    "krk_tanh_norm": [_P, _P, _P, _P, _P, c_float, _P, _P, c_int, c_int, c_int, _P],
     "krk_gated_act": [_P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_float, c_float],
     "krk_hyper_rmsnorm": [_P, _P, _P, _P, _P, _P, _P, c_float, c_int, c_int, c_int, c_float, c_int, _P],
     "krk_bias_row_norm": [_P, c_int, c_int, c_int, c_int, c_int, _P, _P, c_float, c_int, c_int, _P],
     "krk_rotate_norm_write": [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, c_int, c_float, _P, _P,
                               _P, _P, c_int, _P, _P, c_int, c_int, _P, c_int, c_float, c_int, _P],
     "krk_sink_attention": [_P, c_int, c_int, c_float, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P, _P,
-                           c_int, _P, _P, c_int, c_float, c_int, c_int, c_int, _P, c_int, c_int, c_int, c_int, _P],
+                           c_int, _P, _P, c_int, c_int, c_float, c_int, c_int, c_int, _P, c_int, c_int, c_int, c_int, _P],
     "krk_sink_attention_single": [_P, c_int, c_int, c_float, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P,
-                                  c_int, _P, _P, c_int, c_float, c_int, c_int, _P, c_int, c_int, c_int, _P, c_int, c_int, c_float,
+                                  c_int, _P, _P, c_int, c_int, c_float, c_int, c_int, _P, c_int, c_int, c_int, _P, c_int, c_int, c_float,
                                   c_int, c_int, _P, c_int, c_int, c_int, c_int, _P],
     "krk_latent_norm_write": [_P, c_int, c_int, c_int, _P, c_float, _P, _P, _P, _P, c_int, c_int, _P, c_int, _P, c_int, _P],
-    "krk_head_linear": [_P, c_int, c_int, c_float, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P],
+    "krk_head_linear": [_P, c_int, c_int, c_int, c_float, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P, c_float,
+                        _P, _P, c_int, c_int, _P],
+    "krk_latent_rows": [_P, _P, c_int, c_int, c_int, _P, c_int, c_int, _P, c_int, _P, c_float, c_float, _P, _P, _P, _P, c_int,
+                        _P, c_int, c_int, _P],
+    "krk_latent_gather": [_P, _P, c_int, c_int, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P],
     "krk_embed_bigram": [_P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_longlong, c_longlong, _P, _P, _P, _P, _P, c_int, _P],
     "krk_bias_norm_rotate_write": [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_float, _P, c_int,
                                    c_int, _P, _P, _P, _P, c_int, _P, _P, c_int, c_int, c_int, _P],
@@ -80,11 +85,19 @@ _MIX_SIGNATURES = {
 _MOE_SIGNATURES = {
     "krk_moe_route": [_P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, _P, c_int],
     "krk_moe_route_groups": [_P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P],
-    "krk_moe_gate_up_pairs": [_P, _P, c_int, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P],
-    "krk_moe_down_pairs": [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P],
+    "krk_moe_route_softmax_groups": [_P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P],
+    "krk_moe_gate_up_pairs": [_P, _P, c_int, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P],
+    "krk_moe_down_pairs": [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, _P, c_int, _P, c_int, _P],
     "krk_moe_sort": [_P, _P, _P, c_int, c_int, c_int, _P],
     "krk_moe_gather": [_P, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P],
-    "krk_moe_combine": [_P, _P, _P, _P, _P, _P, _P, c_int, _P, c_int, c_int, c_int, c_int, _P],
+    "krk_moe_combine": [_P, _P, _P, _P, _P, _P, _P, c_int, _P, c_int, c_int, c_int, _P, c_int, _P, c_int, _P],
+}
+_MEMORY_SIGNATURES = {
+    "krk_memory_gates": [_P, _P, c_int, _P, c_float, _P, c_int, c_int, c_int, c_int, _P, _P, _P, c_int, _P],
+    "krk_memory_decays": [_P, _P, c_int, _P, _P, c_float, c_int, c_int, c_int, c_int, _P],
+    "krk_memory_scan": [_P, _P, c_int, _P, c_int, _P, c_int, c_float, _P, _P, _P, _P, c_int, c_int, c_int, c_int, _P, _P, _P,
+                        c_int, _P],
+    "krk_memory_finish": [_P, c_int, c_int, c_float, _P, _P, _P, c_int, _P, c_int, c_int, c_float, c_int, c_int, _P],
 }
 _SCAN_SIGNATURES = {
     "krk_token_shift": [_P, _P, c_int, _P, _P, c_int, c_int, c_int, _P, _P, _P, c_int, _P, c_int],
@@ -96,7 +109,7 @@ _SCAN_SIGNATURES = {
                      c_int, _P, _P, _P, c_int, _P, _P, c_int, _P],
     "krk_gated_group_norm": [_P, c_int, c_int, c_float, _P, _P, c_int, _P, c_int, c_int, c_int, c_float, c_int, _P],
 }
-_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "sigmoid": 2, "swish_clamped": 3, "xielu": 4}
+_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "sigmoid": 2, "swish_clamped": 3, "xielu": 4, "relu2": 5}
 _ATTN_SIGNATURES = {
     "krk_attention_simple": [_P, _P, c_int, c_int, c_int, _P, _P, _P, _P, c_int, _P, _P, c_int, c_float, c_int, c_int, _P],
     "krk_attention_head_dim": [],
@@ -147,7 +160,7 @@ class Kernels:
             raise KernelError("no CUDA device: this library computes with its CUDA kernels only")
         self.device = torch.device(device)
         self.core = _load(build_library("core"), _SIGNATURES)
-        self._mix = self._scan = self._moe = None
+        self._mix = self._scan = self._moe = self._memory = None
         self.attn: dict[int, ctypes.CDLL] = {}
         for d in head_dims:
             self._attn_lib(int(d))
@@ -503,6 +516,13 @@ class Kernels:
         return self._scan
 
     @property
+    def memory(self) -> ctypes.CDLL:
+        """The library of the matrix-state mixers without a removal term, compiled and loaded at their first call."""
+        if self._memory is None:
+            self._memory = _load(build_library("memory"), _MEMORY_SIGNATURES)
+        return self._memory
+
+    @property
     def moe(self) -> ctypes.CDLL:
         """The library of the routed-experts kernels, compiled and loaded at their first call."""
         if self._moe is None:
@@ -571,6 +591,22 @@ class Kernels:
                                            self._stream()), "wide rmsnorm")
         return out if gain2 is None else (out, out2)
 
+    def tanh_norm(self, x, branch, fold, alpha, gain, shift, x_new, out_dtype):
+        """tanh(alpha * s) * gain + shift in ``out_dtype`` with s = x (float32), or x + fold * branch, written to ``x_new``
+        (``fold``: a float32 vector, None: 1)."""
+        C = x.shape[1]
+        if x.dtype != torch.float32 or not x.is_contiguous() or any(
+                t is not None and (t.dtype != torch.float32 or t.numel() != C) for t in (gain, shift, fold)):
+            raise KernelError("this norm reads a contiguous float32 stream and float32 vectors of its width")
+        if branch is not None and (branch.dtype != out_dtype or not branch.is_contiguous() or branch.shape != x.shape):
+            raise KernelError("the pending output must have the path's dtype and the stream's shape")
+        out = torch.empty(x.shape, dtype=out_dtype, device=x.device)
+        self._ok(self.mix.krk_tanh_norm(out.data_ptr(), x_new.data_ptr() if branch is not None else None, x.data_ptr(),
+                                        _ptr(branch), _ptr(fold) if branch is not None else None, float(alpha),
+                                        gain.data_ptr(), shift.data_ptr(), x.shape[0], C, _code(out_dtype), self._stream()),
+                 "tanh norm")
+        return out
+
     def gated_act(self, gu, intermediate, activation, row_gate_col=None, act_params=None):
         """act(gu[:, :I]) * gu[:, I:2I], times sigmoid(gu[:, row_gate_col]) per row if that column is given.
         "swish_clamped" takes ``act_params`` = (limit, slope)."""
@@ -617,9 +653,51 @@ class Kernels:
             else:
                 torch.mul(y.transpose(0, 1), out_scale, out=dst)
             return out
-        self._ok(self.mix.krk_head_linear(optr, ostride, int(out_col), float(out_scale), ptr, stride, w.data_ptr(), heads, N,
-                                          K, x.shape[0], _code(x.dtype), self._stream()), "per-head product")
+        self._ok(self.mix.krk_head_linear(optr, ostride, int(out_col), N, float(out_scale), ptr, stride, K, w.data_ptr(), heads,
+                                          N, K, x.shape[0], 0, None, 1.0, None, None, 0, _code(x.dtype), self._stream()),
+                 "per-head product")
         return out
+
+    # -- latent attention with a rotated part ------------------------------------------------
+    def latent_rows(self, proj, query, rows, rot_dim, inv_freq, rot_factor, eps, batch, cache):
+        """``query`` (column, size, gain): those columns of ``proj``, RMS-normed with a float32 gain, are returned. ``rows``
+        (column, rank, gain) or None: that many columns likewise, and behind them ``rot_dim`` columns rotated, go to the
+        positions' places in the cache."""
+        ptr, stride = self._rows_view(proj)
+        q_col, q_size, q_gain = query
+        c_col, rank, c_gain = rows if rows is not None else (0, 0, None)
+        if rows is not None and (cache.k.dtype != proj.dtype or cache.head_dim != rank + rot_dim or cache.kv_heads != 1
+                                 or c_gain.dtype != torch.float32):
+            raise KernelError("the cache does not fit the latent rows it is to receive")
+        out = torch.empty((proj.shape[0], q_size), dtype=proj.dtype, device=proj.device)
+        self._ok(self.mix.krk_latent_rows(out.data_ptr(), ptr, stride, int(q_col), int(q_size), q_gain.data_ptr(), int(c_col),
+                                          int(rank), _ptr(c_gain), int(rot_dim), inv_freq.data_ptr(), float(rot_factor),
+                                          float(eps), batch.row_seq.data_ptr(), batch.row_pos.data_ptr(),
+                                          batch.seq_slot.data_ptr(), cache.table.data_ptr(), cache.width,
+                                          cache.k.data_ptr() if rows is not None else None, proj.shape[0], _code(proj.dtype),
+                                          self._stream()), "low-rank rows")
+        return out
+
+    def rotated_latent_attention(self, q, m, batch, cache, gate, out, out_col, out_scale, shared):
+        """Attention of queries [rows, heads * (dim + rot)] (not rotated yet) over the cached rows [latent | rotated key],
+        times sigmoid of ``gate`` = (rows, first column), into ``out``'s columns. ``m`` gives the sizes and weights
+        (parts/latent_attention.py)."""
+        H, D, E, R, P = m.heads, m.dim, m.rot, m.rank, m.vdim
+        rows = q.shape[0]
+        W = R + E
+        g_ptr, g_stride = self._rows_view(gate[0])
+        g_ptr += int(gate[1]) * gate[0].element_size()
+        optr, ostride = self._rows_view(out)
+        # a head's query is carried into the latent space, attention runs over the cached rows themselves
+        qx = torch.empty((rows, H * W), dtype=q.dtype, device=q.device)
+        self._ok(self.mix.krk_head_linear(qx.data_ptr(), H * W, 0, W, 1.0, q.data_ptr(), q.stride(0), D + E, m.uk_t.data_ptr(), H,
+                                          R, D, rows, E, m.inv_freq.data_ptr(), float(m.rot_factor), batch.row_pos.data_ptr(),
+                                          None, 0, _code(q.dtype), self._stream()), "queries into the latent space")
+        mixed = torch.empty((rows, H * R), dtype=q.dtype, device=q.device)
+        self.sink_attention(qx, 0, H, W, R, None, m.scale, None, batch, cache, mixed, 0, 1.0)
+        self._ok(self.mix.krk_head_linear(optr, ostride, int(out_col), P, float(out_scale), mixed.data_ptr(), H * R, R,
+                                          m.uv.data_ptr(), H, P, R, rows, 0, None, 1.0, None, g_ptr, g_stride, _code(q.dtype),
+                                          self._stream()), "values out of the latent space")
 
     # -- routed experts ------------------------------------------------------------------------
     MOE_PAIR_ROWS = 16  # rows up to which every (row, expert) pair reads its expert's weights by itself
@@ -649,10 +727,36 @@ class Kernels:
                                         rows, E, int(gate_row), int(top), self._stream(), int(over_all)), "expert routing")
         return experts, weights, row_gate
 
+    def moe_route_softmax_groups(self, x, w, correction, top, groups, keep, identity, gate_row=False):
+        """(experts int32 [rows, top], weights float32 [rows, top], row gate or None, passed float32 [rows] or None): softmax
+        scores over all outputs, the choice by score + correction among the outputs of the ``keep`` best of ``groups``
+        groups of neighbours (a group's score: its largest), the weights the chosen scores. The last ``identity`` outputs
+        hand their input through: such a choice is expert -1 with weight 0, and its weight is in ``passed``. ``gate_row`` as
+        in ``moe_route``."""
+        outputs = w.shape[0] - int(gate_row)
+        rows = x.shape[0]
+        if correction.dtype != torch.float32 or correction.numel() != outputs:
+            raise KernelError("the routing correction is one float32 number per output of the router")
+        experts = torch.empty((rows, top), dtype=torch.int32, device=x.device)
+        weights = torch.empty((rows, top), dtype=torch.float32, device=x.device)
+        row_gate = torch.empty(rows, dtype=torch.float32, device=x.device) if gate_row else None
+        passed = torch.empty(rows, dtype=torch.float32, device=x.device) if identity else None
+        logits = self.linear(x, w, out_float32=True)
+        self._ok(self.moe.krk_moe_route_softmax_groups(experts.data_ptr(), weights.data_ptr(), _ptr(row_gate), _ptr(passed),
+                                                       logits.data_ptr(), correction.data_ptr(), rows, outputs,
+                                                       outputs - int(identity), int(gate_row), int(top), int(groups), int(keep),
+                                                       self._stream()), "expert routing by softmax within groups")
+        return experts, weights, row_gate, passed
+
+    def up_act(self, h, w_up, activation):
+        """act(up h), without a gate."""
+        return self.act_rows(self.linear(h, w_up), activation)
+
     def moe_experts(self, x, w_gate_up, w_down, experts, weights, intermediate, activation, add=None, add_gate=None,
-                    batch=None):
-        """add * add_gate + sum_j weights[r, j] * expert_{experts[r, j]}(x[r]); w_gate_up [E, 2F, K], w_down [E, C, F];
-        ``add_gate``: one float32 number per row (None: 1)."""
+                    batch=None, gated=True, add_input=None):
+        """add * add_gate + add_input * x + sum_j weights[r, j] * expert_{experts[r, j]}(x[r]) over the choices that are not
+        -1; w_gate_up [E, 2F, K] ([E, F, K] without ``gated``), w_down [E, C, F]; ``add_gate`` (None: 1) and ``add_input``
+        (None: 0): one float32 number per row."""
         rows, top = experts.shape
         E, C, F = w_down.shape
         K = x.shape[1]
@@ -663,10 +767,11 @@ class Kernels:
         if single or rows * top <= max(self.MOE_PAIR_ROWS * top, 2 * E):
             pairs = torch.empty((rows * top, F), dtype=x.dtype, device=x.device)
             self._ok(self.moe.krk_moe_gate_up_pairs(pairs.data_ptr(), ptr, stride, w_gate_up.data_ptr(), experts.data_ptr(),
-                                                    rows, top, F, K, act, _code(x.dtype), self._stream()), "experts' gate/up")
+                                                    rows, top, F, K, act, int(gated), _code(x.dtype), self._stream()),
+                     "experts' gate/up")
             self._ok(self.moe.krk_moe_down_pairs(out.data_ptr(), _ptr(add), _ptr(add_gate), pairs.data_ptr(), w_down.data_ptr(),
-                                                 experts.data_ptr(), weights.data_ptr(), rows, top, C, F, _code(x.dtype),
-                                                 self._stream()), "experts' down")
+                                                 experts.data_ptr(), weights.data_ptr(), rows, top, C, F, ptr, stride,
+                                                 _ptr(add_input), _code(x.dtype), self._stream()), "experts' down")
             return out
         # many rows: ordered by expert on the device; the experts' row counts come to the host (a step of many
         # tokens is never replayed from a graph)
@@ -688,18 +793,18 @@ class Kernels:
             # bfloat16: every expert's rows start at a multiple of cap (the most rows any expert got), and the
             # library's batched product takes all experts at once; the rows beyond an expert's own are never read back
             gu = torch.bmm(xg.view(E, cap, K), w_gate_up.transpose(1, 2))
-            h = self.gated_act(gu.view(E * cap, 2 * F), F, activation)
+            h = self.gated_act(gu.view(E * cap, 2 * F), F, activation) if gated else self.act_rows(gu.view(E * cap, F), activation)
             yg = torch.bmm(h.view(E, cap, F), w_down.transpose(1, 2)).view(E * cap, C)
         else:
             yg = torch.empty((n_rows, C), dtype=x.dtype, device=x.device)
             for e in range(E):
                 a, b = bounds[e], bounds[e + 1]
                 if b > a:
-                    h = self.gate_up_act(xg[a:b], w_gate_up[e], F, activation)
+                    h = self.gate_up_act(xg[a:b], w_gate_up[e], F, activation) if gated else self.up_act(xg[a:b], w_gate_up[e], activation)
                     yg[a:b] = self.linear(h, w_down[e])
         self._ok(self.moe.krk_moe_combine(out.data_ptr(), _ptr(add), _ptr(add_gate), yg.data_ptr(), place.data_ptr(), experts.data_ptr(),
-                                          offsets.data_ptr(), cap, weights.data_ptr(), rows, top, C, _code(x.dtype),
-                                          self._stream()), "experts' sum")
+                                          offsets.data_ptr(), cap, weights.data_ptr(), rows, top, C, ptr, stride,
+                                          _ptr(add_input), _code(x.dtype), self._stream()), "experts' sum")
         return out
 
     def gate_up_act(self, h, w_gate_up, intermediate, activation, act_params=None):
@@ -777,7 +882,7 @@ class Kernels:
             rc = self.mix.krk_sink_attention_single(
                 optr, ostride, out_col, float(out_scale), ptr, stride, q_col, heads, cache.kv_heads, dim, vdim,
                 _ptr(sink), batch.seq_slot.data_ptr(), batch.seq_start.data_ptr(), cache.table.data_ptr(), cache.width,
-                cache.k.data_ptr(), cache.v.data_ptr(), batch.n_seqs, float(scale), int(window or 0), splits,
+                cache.k.data_ptr(), cache.v.data_ptr(), cache.v_dim, batch.n_seqs, float(scale), int(window or 0), splits,
                 _ptr(scratch), *((1, fuse[0], fuse[1], fuse[2].data_ptr(), fuse[3], int(fuse[4] is not None),
                                   float(fuse[4] or 0.0)) if fuse else (0, 0, 0, None, 0, 0, 0.0)),
                 *extras, _code(proj.dtype), self._stream())
@@ -788,7 +893,7 @@ class Kernels:
                 return False
         elif fuse:
             return False
-        if (proj.dtype == torch.bfloat16 and dim == vdim and dim % 16 == 0 and dim <= 256 and dim in self.attn
+        if (proj.dtype == torch.bfloat16 and dim == vdim == cache.v_dim and dim % 16 == 0 and dim <= 256 and dim in self.attn
                 and not batch.is_decode and hasattr(self.attn[dim], "krk_sink_window_prefill")):
             # many tokens per sequence in bfloat16: the tensor-core walk over whole pages (compiled per head size)
             esz = proj.element_size()
@@ -804,7 +909,7 @@ class Kernels:
         self._ok(self.mix.krk_sink_attention(
             optr, ostride, out_col, float(out_scale), ptr, stride, q_col, heads, cache.kv_heads, dim, vdim, _ptr(sink),
             batch.row_seq.data_ptr(), batch.row_pos.data_ptr(), batch.seq_slot.data_ptr(), cache.table.data_ptr(),
-            cache.width, cache.k.data_ptr(), cache.v.data_ptr(), proj.shape[0], float(scale), int(window or 0),
+            cache.width, cache.k.data_ptr(), cache.v.data_ptr(), cache.v_dim, proj.shape[0], float(scale), int(window or 0),
             *extras, _code(proj.dtype), self._stream()), "windowed attention with a sink")
 
     # -- pair-hash embedding, per-head norms with pair rotation, mixed head scores over blocks of keys ------------
@@ -977,6 +1082,48 @@ class Kernels:
             lora.shape[1], batch.n_seqs, batch.cu_q.data_ptr(), batch.seq_qlen.data_ptr(), batch.seq_slot.data_ptr(),
             rows, _ptr(prep), _ptr(o_raw), _code(r.dtype), self._stream())
         self._ok(rc, f"{kind} recurrence (heads of up to 256 channels)")
+
+    # -- matrix states without a removal term -------------------------------------------------
+    def _memory_scan(self, q, k, v, gate, decays, gates, heads, dim, vdim, norm_w, eps, state, nm, batch, out, out_col, out_scale):
+        views = [self._rows_view(t) for t in (q, k, v, gate)]
+        optr, ostride = self._rows_view(out)
+        rows = q.shape[0]
+        if state.dtype != torch.float32 or not state.is_contiguous() or state.shape[1:] != (heads, dim, vdim):
+            raise KernelError("the scan keeps a contiguous float32 state [slots, heads, dim, vdim]")
+        if nm is not None and (nm.dtype != torch.float32 or not nm.is_contiguous() or nm.shape[1:] != (heads, dim + 1)):
+            raise KernelError("the gated scan keeps a contiguous float32 [slots, heads, dim + 1] beside its state")
+        y = torch.empty((rows, heads * (vdim + int(nm is not None))), dtype=torch.float32, device=q.device)
+        self._ok(self.memory.krk_memory_scan(y.data_ptr(), *views[0], *views[1], *views[2], float(dim) ** -0.5, _ptr(decays),
+                                             _ptr(gates), state.data_ptr(), _ptr(nm), heads, dim, vdim, batch.n_seqs,
+                                             batch.cu_q.data_ptr(), batch.seq_qlen.data_ptr(), batch.seq_slot.data_ptr(),
+                                             _code(q.dtype), self._stream()), "matrix-state scan (up to 1,024 key channels a head)")
+        self._ok(self.memory.krk_memory_finish(optr, ostride, int(out_col), float(out_scale), y.data_ptr(), _ptr(gates), *views[3],
+                                               norm_w.data_ptr(), heads, vdim, float(eps), rows, _code(q.dtype), self._stream()),
+                 "matrix-state head norm and gate")
+
+    def gla_scan(self, q, k, v, gate, lora, w2, bias, tau, heads, dim, vdim, norm_w, eps, state, batch, out, out_col, out_scale):
+        """Gated linear attention over a step's rows, from and to ``state`` [slots, heads, dim, vdim]; see
+        csrc/matrix_memory.cu. ``norm_w`` [vdim]."""
+        lptr, lstride = self._rows_view(lora)
+        rows, R = lora.shape
+        if w2.dtype != q.dtype or not w2.is_contiguous() or bias.dtype != torch.float32:
+            raise KernelError("the decays read their second matrix in the path's dtype and a float32 bias")
+        decays = torch.empty((rows, heads * dim), dtype=torch.float32, device=q.device)
+        self._ok(self.memory.krk_memory_decays(decays.data_ptr(), lptr, lstride, w2.data_ptr(), bias.data_ptr(), float(tau), rows,
+                                               heads * dim, R, _code(q.dtype), self._stream()), "log decays")
+        self._memory_scan(q, k, v, gate, decays, None, heads, dim, vdim, norm_w, eps, state, None, batch, out, out_col, out_scale)
+
+    def mlstm_scan(self, q, k, v, gate, if_rows, if_bias, cap, heads, dim, vdim, norm_w, eps, state, nm, batch, out, out_col,
+                   out_scale):
+        """The matrix LSTM over a step's rows; ``if_rows`` [rows, 2 * heads]: input then forget gates before bias and cap;
+        ``nm`` [slots, heads, dim + 1]: the vector beside the matrix and the running maximum. ``norm_w`` [heads * vdim]."""
+        zptr, zstride = self._rows_view(if_rows)
+        rows = q.shape[0]
+        gates = torch.empty((rows, heads, 4), dtype=torch.float32, device=q.device)
+        self._ok(self.memory.krk_memory_gates(gates.data_ptr(), zptr, zstride, if_bias.data_ptr(), float(cap), nm.data_ptr(), heads,
+                                              dim, batch.n_seqs, batch.max_q_len, batch.cu_q.data_ptr(), batch.seq_qlen.data_ptr(),
+                                              batch.seq_slot.data_ptr(), _code(q.dtype), self._stream()), "matrix LSTM gates")
+        self._memory_scan(q, k, v, gate, None, gates, heads, dim, vdim, norm_w, eps, state, nm, batch, out, out_col, out_scale)
 
     # -- state-space mixer ------------------------------------------------------------------
     SSD_CHUNK = 128  # tokens per chunk where one sequence's step is long enough to be scanned in chunks

@@ -4,8 +4,9 @@ Kinds of library: ``core`` (kernels whose sizes are run-time arguments),
 ``attn_d<D>`` (the attention kernels, compiled once per head size D with
 ``-DKRK_HEAD_DIM=D``, so a model compiles only the head size it has), ``mix``
 (the kernels of models with a 32-bit residual stream, windowed attention with a
-sink or over latent rows), ``scan`` (recurrent state) and ``moe`` (routed
-experts); each of the last three is compiled and loaded when a model first calls
+sink or over latent rows), ``scan`` (recurrent state), ``memory`` (matrix states
+without a removal term) and ``moe`` (routed
+experts); each of the last four is compiled and loaded when a model first calls
 one of its kernels, so a model compiles what it needs. A library
 is rebuilt when a source or a flag changes (its name carries a hash of both) and
 is otherwise loaded as it is. Libraries live in ``csrc/_build`` inside the
@@ -34,8 +35,9 @@ CORE_SOURCES = ["elementwise.cu", "rope_kv.cu", "gemm_simple.cu", "select.cu", "
 CORE_LIBS = ["-lcublasLt"]  # lt_gemm.cu; the process already holds the copy that torch loaded
 MIX_SOURCES = ["wide_rows.cu", "sink_attention.cu", "latent.cu", "hyper.cu", "mixed_attention.cu"]
 SCAN_SOURCES = ["recurrent.cu", "ssd.cu"]
+MEMORY_SOURCES = ["matrix_memory.cu"]
 MOE_SOURCES = ["routed.cu"]
-SMALL_LIBRARIES = {"mix": MIX_SOURCES, "scan": SCAN_SOURCES, "moe": MOE_SOURCES}
+SMALL_LIBRARIES = {"mix": MIX_SOURCES, "scan": SCAN_SOURCES, "memory": MEMORY_SOURCES, "moe": MOE_SOURCES}
 ATTN_SOURCES = ["attention_simple.cu", "attention_mma.cu", "attention_tcgen05.cu"]
 HEADERS = ["common.cuh", "mma.cuh", "tcgen05.cuh", "attention_noalloc.h"]
 

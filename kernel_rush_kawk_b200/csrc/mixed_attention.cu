@@ -479,10 +479,11 @@ __global__ void norm_sum_kernel(T* __restrict__ out, NormSumArgs a, int C, float
 __device__ __forceinline__ float act_value(float v, int act, float pa, float pb) {
   if (act == 4) return v > 0.f ? pa * v * v + 0.5f * v : pb * (expm1f(v) - v) + 0.5f * v;
   if (act == 1) return 0.5f * v * (1.0f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
+  if (act == 5) return v > 0.f ? v * v : 0.f;
   return v / (1.0f + expf(-v));
 }
 
-// act 0: silu, 1: tanh-GELU, 4: xIELU with pa = softplus(p), pb = 1/2 + softplus(q). One block row (blockIdx.y) and
+// act 0: silu, 1: tanh-GELU, 4: xIELU with pa = softplus(p), pb = 1/2 + softplus(q), 5: squared relu. One block row (blockIdx.y) and
 // column chunk; V elements (16 bytes) a thread at a time where the row allows it.
 template <typename T, int V>
 __global__ void act_rows_kernel(T* __restrict__ out, const T* __restrict__ z, int z_stride, int I, int act, float pa,
@@ -644,7 +645,7 @@ KRK_API int krk_norm_sum(void* out, const void* y0, const void* y1, const void* 
 KRK_API int krk_act_rows(void* out, const void* z, int z_stride, int rows, int I, int act, float pa, float pb, int dtype,
                          cudaStream_t stream) {
   if (rows == 0 || I == 0) return 0;
-  if ((act != 0 && act != 1 && act != 4) || rows > 65535 * 16) return -2;
+  if ((act != 0 && act != 1 && act != 4 && act != 5) || rows > 65535 * 16) return -2;
   const int V = dtype == KRK_DTYPE_F32 ? 4 : 8;
   const bool vec = I % V == 0 && z_stride % V == 0 && (((uintptr_t)out | (uintptr_t)z) & 15) == 0;
   const int pieces = vec ? I / V : I;

@@ -9,7 +9,11 @@
 // against 1.53 ms a step of one sequence at 64 experts of width 2,048.)
 //
 // krk_moe_route_groups: the same walk over other scores (sigmoid scores, a stored correction for the choice, groups of
-// experts of which only the best may be chosen); see moe_route_groups_kernel.
+// experts of which only the best may be chosen; or softmax scores, see krk_moe_route_softmax_groups); see
+// moe_route_groups_kernel. There the last outputs of the router may be identity experts, which hand the token's row
+// through: such a choice is left out of the experts' work (expert number -1, weight 0), and the sum of the row's
+// identity weights goes to a buffer of its own; whoever adds up the experts' results also adds that number times the
+// row. Every kernel below takes -1 for "no expert".
 //
 // Few rows (single-token steps): a (row, chosen expert) pair reads its expert's weights once.
 //   krk_moe_gate_up_pairs: act[pair, f] = a(Wg_e[f] . x_r) * (Wu_e[f] . x_r), a warp per f, lanes over K.
@@ -28,6 +32,7 @@ namespace {
 __device__ __forceinline__ float act_of(float z, int act) {
   if (act == 0) return z / (1.0f + expf(-z));
   if (act == 1) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  if (act == 5) return z > 0.f ? z * z : 0.f;
   return 1.0f / (1.0f + expf(-z));
 }
 
@@ -113,9 +118,13 @@ __device__ __forceinline__ void warp_argmax(const float* z, int n, int lane, flo
 // Sigmoid scores chosen within the best groups: s = sigmoid(logit); the choice goes by c = s + correction; the experts
 // are `groups` equal runs of neighbours, a group's score is the sum of its two largest c (its one c where a group has one
 // expert), only the `keep` best groups' experts can be chosen; the weights are the chosen s / (their sum + 1e-20) * scale.
+// SOFTMAX: s = softmax of the logits over all E outputs, a group's score is its one largest c, the weights are the chosen s
+// as they are, and a chosen output from `real` on is an identity expert.
+template <bool SOFTMAX>
 __global__ void moe_route_groups_kernel(int* __restrict__ experts, float* __restrict__ weights, float* __restrict__ row_gate,
                                         const float* __restrict__ logits, const float* __restrict__ correction, int rows,
-                                        int E, int has_gate, int top, int groups, int keep, float scale) {
+                                        int E, int has_gate, int top, int groups, int keep, float scale, int real,
+                                        float* __restrict__ passed) {
   extern __shared__ float z_s[];  // [warps][2 E + 2 groups]
   grid_launch_dependents();
   grid_dependency_wait();
@@ -127,8 +136,17 @@ __global__ void moe_route_groups_kernel(int* __restrict__ experts, float* __rest
   float* gs = s + E;
   int* kept = reinterpret_cast<int*>(gs + groups);
   const float* src = logits + (size_t)row * (E + has_gate);
+  float big = 0.f, inv = 1.f;
+  if (SOFTMAX) {
+    big = -INFINITY;
+    for (int e = lane; e < E; e += 32) big = fmaxf(big, src[e]);
+    big = warp_max(big);
+    float all = 0.f;
+    for (int e = lane; e < E; e += 32) all += expf(src[e] - big);
+    inv = 1.0f / warp_sum(all);
+  }
   for (int e = lane; e < E; e += 32) {
-    const float v = act_of(src[e], 2);
+    const float v = SOFTMAX ? expf(src[e] - big) * inv : act_of(src[e], 2);
     s[e] = v;
     c[e] = v + correction[e];
   }
@@ -143,7 +161,7 @@ __global__ void moe_route_groups_kernel(int* __restrict__ experts, float* __rest
         if (v > a) { b = a; a = v; }
         else if (v > b) b = v;
       }
-      gs[g] = size > 1 ? a + b : a;
+      gs[g] = (!SOFTMAX && size > 1) ? a + b : a;
       kept[g] = 0;
     }
     __syncwarp();
@@ -174,6 +192,16 @@ __global__ void moe_route_groups_kernel(int* __restrict__ experts, float* __rest
     if (lane == 0) c[best_e] = -INFINITY;
     __syncwarp();
   }
+  if (SOFTMAX) {
+    const bool identity = lane < top && mine_e >= real;
+    const float handed = warp_sum(identity ? mine : 0.f);
+    if (passed && lane == 0) passed[row] = handed;
+    if (lane < top) {
+      experts[(size_t)row * top + lane] = identity ? -1 : mine_e;
+      weights[(size_t)row * top + lane] = identity ? 0.f : mine;
+    }
+    return;
+  }
   if (lane < top) {
     experts[(size_t)row * top + lane] = mine_e;
     weights[(size_t)row * top + lane] = mine / (total + 1e-20f) * scale;
@@ -185,17 +213,25 @@ constexpr int PAIR_WARPS = 8;
 template <typename T>
 __global__ void __launch_bounds__(PAIR_WARPS * 32)
 moe_gate_up_pairs_kernel(T* __restrict__ act_out, const T* __restrict__ x, int x_stride, const T* __restrict__ w,
-                         const int* __restrict__ experts, int top, int F, int K, int act) {
+                         const int* __restrict__ experts, int top, int F, int K, int act, int gated) {
   extern __shared__ __align__(16) float xs[];  // [K]
   grid_launch_dependents();
   grid_dependency_wait();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int pair = blockIdx.y;
   const int e = experts[pair];
+  if (e < 0) return;
   const T* xr = x + (size_t)(pair / top) * x_stride;
   for (int k = threadIdx.x; k < K; k += blockDim.x) xs[k] = to_float<T>(xr[k]);
   __syncthreads();
-  const T* we = w + (size_t)e * 2 * F * K;
+  const T* we = w + (size_t)e * (gated ? 2 : 1) * F * K;
+  if (!gated) {
+    for (int f = blockIdx.x * PAIR_WARPS + warp; f < F; f += gridDim.x * PAIR_WARPS) {
+      const float u = warp_sum(lane_dot<T>(we + (size_t)f * K, xs, K, lane));
+      if (lane == 0) act_out[(size_t)pair * F + f] = from_float<T>(act_of(round_to<T>(u), act));
+    }
+    return;
+  }
   for (int f = blockIdx.x * PAIR_WARPS + warp; f < F; f += gridDim.x * PAIR_WARPS) {
     const T* wg = we + (size_t)f * K;
     const T* wu = we + (size_t)(F + f) * K;
@@ -210,33 +246,39 @@ template <typename T>
 __global__ void __launch_bounds__(PAIR_WARPS * 32)
 moe_down_pairs_kernel(T* __restrict__ out, const T* __restrict__ add, const float* __restrict__ add_gate, const T* __restrict__ act_in,
                       const T* __restrict__ w, const int* __restrict__ experts, const float* __restrict__ weights, int top,
-                      int C, int F) {
+                      int C, int F, const T* __restrict__ x, int x_stride, const float* __restrict__ passed) {
   extern __shared__ __align__(16) float as[];  // [top][F4], F4 = F rounded up to a multiple of 4
   const int F4 = (F + 3) & ~3;
   grid_launch_dependents();
   grid_dependency_wait();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int row = blockIdx.y;
-  for (int i = threadIdx.x; i < top * F; i += blockDim.x) as[(i / F) * F4 + i % F] = to_float<T>(act_in[(size_t)row * top * F + i]);
+  // an absent expert's activations were never written: zeros
+  for (int i = threadIdx.x; i < top * F; i += blockDim.x)
+    as[(i / F) * F4 + i % F] = experts[(size_t)row * top + i / F] < 0 ? 0.f : to_float<T>(act_in[(size_t)row * top * F + i]);
   __syncthreads();
   for (int c = blockIdx.x * PAIR_WARPS + warp; c < C; c += gridDim.x * PAIR_WARPS) {
     float total = add ? to_float<T>(add[(size_t)row * C + c]) * (add_gate ? add_gate[row] : 1.f) : 0.f;
+    if (passed) total += passed[row] * to_float<T>(x[(size_t)row * x_stride + c]);
     // four experts' rows are read side by side, so that four times the bytes are in flight; the results are still
     // added in the order of the choice
     for (int j0 = 0; j0 < top; j0 += 4) {
       const T* wr[4];
       float s[4];
+      bool on[4];
 #pragma unroll
       for (int jj = 0; jj < 4; ++jj) {
-        const int j = min(j0 + jj, top - 1);
-        wr[jj] = w + ((size_t)experts[(size_t)row * top + j] * C + c) * F;
+        const int e = experts[(size_t)row * top + min(j0 + jj, top - 1)];
+        on[jj] = e >= 0 && j0 + jj < top;
+        wr[jj] = w + ((size_t)max(e, 0) * C + c) * F;
         s[jj] = 0.f;
       }
       if (sizeof(T) == 2 && (F & 7) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0) {
         for (int k = lane * 8; k < F; k += 256) {
           uint4 raw[4];
 #pragma unroll
-          for (int jj = 0; jj < 4; ++jj) raw[jj] = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(wr[jj]) + k);
+          for (int jj = 0; jj < 4; ++jj)
+            raw[jj] = on[jj] ? *reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(wr[jj]) + k) : make_uint4(0u, 0u, 0u, 0u);
 #pragma unroll
           for (int jj = 0; jj < 4; ++jj) {
             const float* xs = as + min(j0 + jj, top - 1) * F4 + k;
@@ -248,12 +290,13 @@ moe_down_pairs_kernel(T* __restrict__ out, const T* __restrict__ add, const floa
         }
       } else {
 #pragma unroll
-        for (int jj = 0; jj < 4; ++jj) s[jj] = lane_dot<T>(wr[jj], as + min(j0 + jj, top - 1) * F4, F, lane);
+        for (int jj = 0; jj < 4; ++jj)
+          if (on[jj]) s[jj] = lane_dot<T>(wr[jj], as + min(j0 + jj, top - 1) * F4, F, lane);
       }
 #pragma unroll
       for (int jj = 0; jj < 4; ++jj) {
         const float r = warp_sum(s[jj]);
-        if (j0 + jj < top) total += weights[(size_t)row * top + j0 + jj] * round_to<T>(r);
+        if (on[jj]) total += weights[(size_t)row * top + j0 + jj] * round_to<T>(r);
       }
     }
     if (lane == 0) out[(size_t)row * C + c] = from_float<T>(total);
@@ -268,7 +311,8 @@ __global__ void moe_sort_kernel(int* __restrict__ offsets, int* __restrict__ pla
   grid_dependency_wait();
   for (int e = threadIdx.x; e <= E; e += blockDim.x) cnt[e] = 0;
   __syncthreads();
-  for (int i = threadIdx.x; i < pairs; i += blockDim.x) atomicAdd(&cnt[experts[i] + 1], 1);
+  for (int i = threadIdx.x; i < pairs; i += blockDim.x)
+    if (experts[i] >= 0) atomicAdd(&cnt[experts[i] + 1], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     for (int e = 0; e < E; ++e) cnt[e + 1] += cnt[e];
@@ -291,8 +335,9 @@ __global__ void moe_sort_kernel(int* __restrict__ offsets, int* __restrict__ pla
 
 __device__ __forceinline__ int row_of_pair(const int* __restrict__ place, const int* __restrict__ experts,
                                            const int* __restrict__ offsets, int cap, int pair) {
-  if (cap <= 0) return place[pair];
   const int e = experts[pair];
+  if (e < 0) return -1;
+  if (cap <= 0) return place[pair];
   return e * cap + place[pair] - offsets[e];
 }
 
@@ -302,7 +347,9 @@ __global__ void moe_gather_kernel(T* __restrict__ xg, const T* __restrict__ x, i
   grid_dependency_wait();
   const int pair = blockIdx.x;
   const T* src = x + (size_t)(pair / top) * x_stride;
-  T* dst = xg + (size_t)row_of_pair(place, experts, offsets, cap, pair) * K;
+  const int at = row_of_pair(place, experts, offsets, cap, pair);
+  if (at < 0) return;
+  T* dst = xg + (size_t)at * K;
   if ((K * sizeof(T)) % 16 == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0) {
     const int n = K * (int)sizeof(T) / 16;
     for (int k = threadIdx.x; k < n; k += blockDim.x) reinterpret_cast<uint4*>(dst)[k] = reinterpret_cast<const uint4*>(src)[k];
@@ -315,7 +362,7 @@ template <typename T>
 __global__ void moe_combine_kernel(T* __restrict__ out, const T* __restrict__ add, const float* __restrict__ add_gate, const T* __restrict__ yg,
                                    const int* __restrict__ place, const int* __restrict__ experts,
                                    const int* __restrict__ offsets, int cap, const float* __restrict__ weights, int top,
-                                   int C) {
+                                   int C, const T* __restrict__ x, int x_stride, const float* __restrict__ passed) {
   __shared__ int src_row[32];
   __shared__ float src_w[32];
   grid_dependency_wait();
@@ -327,7 +374,9 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const T* __restrict__ ad
   __syncthreads();
   for (int c = threadIdx.x; c < C; c += blockDim.x) {
     float total = add ? to_float<T>(add[(size_t)row * C + c]) * (add_gate ? add_gate[row] : 1.f) : 0.f;
-    for (int j = 0; j < top; ++j) total += src_w[j] * to_float<T>(yg[(size_t)src_row[j] * C + c]);
+    if (passed) total += passed[row] * to_float<T>(x[(size_t)row * x_stride + c]);
+    for (int j = 0; j < top; ++j)
+      if (src_row[j] >= 0) total += src_w[j] * to_float<T>(yg[(size_t)src_row[j] * C + c]);
     out[(size_t)row * C + c] = from_float<T>(total);
   }
 }
@@ -353,12 +402,28 @@ KRK_API int krk_moe_route_groups(int* experts, float* weights, float* row_gate, 
     return -2;
   const size_t smem = (size_t)ROUTE_WARPS * (2 * E + 2 * groups) * sizeof(float);
   if (smem > 48 * 1024) return -2;
-  return (int)launch_pdl(moe_route_groups_kernel, dim3((rows + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem,
-                         stream, experts, weights, row_gate, logits, correction, rows, E, has_gate, top, groups, keep, scale);
+  return (int)launch_pdl(moe_route_groups_kernel<false>, dim3((rows + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem,
+                         stream, experts, weights, row_gate, logits, correction, rows, E, has_gate, top, groups, keep, scale, E, (float*)nullptr);
+}
+
+// logits [rows, E + has_gate] over experts and identity experts together; outputs `real`.. are identity experts; passed
+// [rows] (may be null where there are none): the sum of the row's identity weights
+KRK_API int krk_moe_route_softmax_groups(int* experts, float* weights, float* row_gate, float* passed, const float* logits,
+                                         const float* correction, int rows, int E, int real, int has_gate, int top, int groups,
+                                         int keep, cudaStream_t stream) {
+  if (rows == 0) return 0;
+  if (top < 1 || top > 32 || top > E || groups < 1 || E % groups || keep < 1 || keep > groups || top > keep * (E / groups) ||
+      real < 1 || real > E || (real < E && !passed))
+    return -2;
+  const size_t smem = (size_t)ROUTE_WARPS * (2 * E + 2 * groups) * sizeof(float);
+  if (smem > 48 * 1024) return -2;
+  return (int)launch_pdl(moe_route_groups_kernel<true>, dim3((rows + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32),
+                         smem, stream, experts, weights, row_gate, logits, correction, rows, E, has_gate, top, groups, keep, 1.f,
+                         real, passed);
 }
 
 KRK_API int krk_moe_gate_up_pairs(void* act_out, const void* x, int x_stride, const void* w, const int* experts, int rows,
-                                  int top, int F, int K, int act, int dtype, cudaStream_t stream) {
+                                  int top, int F, int K, int act, int gated, int dtype, cudaStream_t stream) {
   if (rows == 0) return 0;
   const size_t smem = (size_t)K * sizeof(float);
   if (smem > 200 * 1024 || (long long)rows * top > 65535) return -2;
@@ -369,13 +434,14 @@ KRK_API int krk_moe_gate_up_pairs(void* act_out, const void* x, int x_stride, co
   const dim3 grid((unsigned)min((F + PAIR_WARPS - 1) / PAIR_WARPS, 1024), (unsigned)(rows * top));
   if (dtype == KRK_DTYPE_F32)
     return (int)launch_pdl(moe_gate_up_pairs_kernel<float>, grid, dim3(PAIR_WARPS * 32), smem, stream, (float*)act_out,
-                           (const float*)x, x_stride, (const float*)w, experts, top, F, K, act);
+                           (const float*)x, x_stride, (const float*)w, experts, top, F, K, act, gated);
   return (int)launch_pdl(moe_gate_up_pairs_kernel<bf16>, grid, dim3(PAIR_WARPS * 32), smem, stream, (bf16*)act_out,
-                         (const bf16*)x, x_stride, (const bf16*)w, experts, top, F, K, act);
+                         (const bf16*)x, x_stride, (const bf16*)w, experts, top, F, K, act, gated);
 }
 
 KRK_API int krk_moe_down_pairs(void* out, const void* add, const float* add_gate, const void* act_in, const void* w, const int* experts,
-                               const float* weights, int rows, int top, int C, int F, int dtype, cudaStream_t stream) {
+                               const float* weights, int rows, int top, int C, int F, const void* x, int x_stride,
+                               const float* passed, int dtype, cudaStream_t stream) {
   if (rows == 0) return 0;
   const size_t smem = (size_t)top * ((F + 3) & ~3) * sizeof(float);
   if (smem > 200 * 1024 || rows > 65535) return -2;
@@ -386,9 +452,9 @@ KRK_API int krk_moe_down_pairs(void* out, const void* add, const float* add_gate
   const dim3 grid((unsigned)min((C + PAIR_WARPS - 1) / PAIR_WARPS, 1024), (unsigned)rows);
   if (dtype == KRK_DTYPE_F32)
     return (int)launch_pdl(moe_down_pairs_kernel<float>, grid, dim3(PAIR_WARPS * 32), smem, stream, (float*)out,
-                           (const float*)add, add_gate, (const float*)act_in, (const float*)w, experts, weights, top, C, F);
+                           (const float*)add, add_gate, (const float*)act_in, (const float*)w, experts, weights, top, C, F, (const float*)x, x_stride, passed);
   return (int)launch_pdl(moe_down_pairs_kernel<bf16>, grid, dim3(PAIR_WARPS * 32), smem, stream, (bf16*)out,
-                         (const bf16*)add, add_gate, (const bf16*)act_in, (const bf16*)w, experts, weights, top, C, F);
+                         (const bf16*)add, add_gate, (const bf16*)act_in, (const bf16*)w, experts, weights, top, C, F, (const bf16*)x, x_stride, passed);
 }
 
 KRK_API int krk_moe_sort(int* offsets, int* place, const int* experts, int rows, int top, int E, cudaStream_t stream) {
@@ -409,13 +475,13 @@ KRK_API int krk_moe_gather(void* xg, const void* x, int x_stride, const int* pla
 }
 
 KRK_API int krk_moe_combine(void* out, const void* add, const float* add_gate, const void* yg, const int* place, const int* experts,
-                            const int* offsets, int cap, const float* weights, int rows, int top, int C, int dtype,
-                            cudaStream_t stream) {
+                            const int* offsets, int cap, const float* weights, int rows, int top, int C, const void* x, int x_stride,
+                            const float* passed, int dtype, cudaStream_t stream) {
   if (rows == 0) return 0;
   if (top > 32) return -2;
   if (dtype == KRK_DTYPE_F32)
     return (int)launch_pdl(moe_combine_kernel<float>, dim3(rows), dim3(256), 0, stream, (float*)out, (const float*)add, add_gate,
-                           (const float*)yg, place, experts, offsets, cap, weights, top, C);
+                           (const float*)yg, place, experts, offsets, cap, weights, top, C, (const float*)x, x_stride, passed);
   return (int)launch_pdl(moe_combine_kernel<bf16>, dim3(rows), dim3(256), 0, stream, (bf16*)out, (const bf16*)add, add_gate,
-                         (const bf16*)yg, place, experts, offsets, cap, weights, top, C);
+                         (const bf16*)yg, place, experts, offsets, cap, weights, top, C, (const bf16*)x, x_stride, passed);
 }

@@ -27,7 +27,8 @@
 // windowed query may also see the first `keep_first` keys (they are walked before the window's own, in position
 // order); the result may be multiplied by sigmoid(gate), one number per head (mode 1) or per element (mode 2),
 // read from the columns `gate_col` of `gate`'s rows; the values that are written may be blended with another
-// layer's values of the same rows, (1 - lambda) v + lambda v_first.
+// layer's values of the same rows, (1 - lambda) v + lambda v_first. A value row of the cache may be wider than the value
+// head (`VP` elements from one to the next, DV of them read): a latent row with a rotated key part behind it.
 #include "common.cuh"
 
 namespace {
@@ -142,7 +143,7 @@ __global__ void sink_attention_kernel(T* __restrict__ out, int out_stride, int o
                                       const float* __restrict__ sink, const int* __restrict__ row_seq,
                                       const int* __restrict__ row_pos, const int* __restrict__ seq_slot,
                                       const int* __restrict__ table, int width, const T* __restrict__ k_cache,
-                                      const T* __restrict__ v_cache, int rows, float scale, int window, int keep_first,
+                                      const T* __restrict__ v_cache, int VP, int rows, float scale, int window, int keep_first,
                                       int keep_pages, const T* __restrict__ gate, int gate_stride, int gate_col,
                                       int gate_mode) {
   extern __shared__ float q_s[];  // warps x D
@@ -192,7 +193,7 @@ __global__ void sink_attention_kernel(T* __restrict__ out, int out_stride, int o
       const float pj = __shfl_sync(0xffffffffu, p, j);
       const int kj = base + j;
       const int page = __shfl_sync(0xffffffffu, my_page, j);  // lane j looked its key's page up already
-      const T* vp = v_cache + (((size_t)page * HKV + kh) * KRK_PAGE + (kj % KRK_PAGE)) * DV;
+      const T* vp = v_cache + (((size_t)page * HKV + kh) * KRK_PAGE + (kj % KRK_PAGE)) * VP;
 #pragma unroll
       for (int i = 0; i < VPL; ++i) {
         const int d = lane + 32 * i;
@@ -251,7 +252,7 @@ sink_attention_single_kernel(T* __restrict__ out, int out_stride, int out_col, f
                              const T* __restrict__ proj, int stride, int q_col, int HQ, int HKV, int D, int DV,
                              const float* __restrict__ sink, const int* __restrict__ seq_slot,
                              const int* __restrict__ seq_start, const int* __restrict__ table, int width,
-                             const T* __restrict__ k_cache, const T* __restrict__ v_cache, float scale, int window,
+                             const T* __restrict__ k_cache, const T* __restrict__ v_cache, int VP, float scale, int window,
                              int SPL, float* __restrict__ scratch, int k_col, int v_col,
                              const float* __restrict__ inv_freq, int rot, int value_norm, float eps, T* k_cache_w,
                              T* v_cache_w, int keep_first, int keep_pages, const T* __restrict__ gate, int gate_stride,
@@ -413,7 +414,7 @@ sink_attention_single_kernel(T* __restrict__ out, int out_stride, int out_col, f
         const int j = j0 + jj;
         const int kj = base + j;
         const int page = __shfl_sync(0xffffffffu, my_page, j & 31);  // lane j looked its key's page up already
-        const T* vp = (FUSE && kj == pos) ? vn : v_cache + (((size_t)page * HKV + kh) * KRK_PAGE + (kj % KRK_PAGE)) * DV;
+        const T* vp = (FUSE && kj == pos) ? vn : v_cache + (((size_t)page * HKV + kh) * KRK_PAGE + (kj % KRK_PAGE)) * VP;
         if (V4) {  // four neighbouring elements per lane, one load
 #pragma unroll
           for (int cb = 0; cb < NV / 4; ++cb)
@@ -563,7 +564,7 @@ KRK_API int krk_rotate_norm_write(void* proj, int stride, int q_col, int k_col, 
 KRK_API int krk_sink_attention(void* out, int out_stride, int out_col, float out_scale, const void* proj, int stride,
                                int q_col, int HQ, int HKV, int D, int DV, const float* sink, const int* row_seq,
                                const int* row_pos, const int* seq_slot, const int* table, int width, const void* k_cache,
-                               const void* v_cache, int rows, float scale, int window, int keep_first, int keep_pages,
+                               const void* v_cache, int v_pitch, int rows, float scale, int window, int keep_first, int keep_pages,
                                const void* gate, int gate_stride, int gate_col, int gate_mode, int dtype,
                                cudaStream_t stream) {
   if (rows == 0) return 0;
@@ -578,11 +579,11 @@ KRK_API int krk_sink_attention(void* out, int out_stride, int out_col, float out
     return (int)launch_pdl(wide ? sink_attention_kernel<float, WIDE_V_PER_LANE> : sink_attention_kernel<float, MAX_V_PER_LANE>, dim3((unsigned)blocks), dim3(warps * 32), smem, stream,
                            (float*)out, out_stride, out_col, out_scale, (const float*)proj, stride, q_col, HQ, HKV, D, DV,
                            sink, row_seq, row_pos, seq_slot, table, width, (const float*)k_cache, (const float*)v_cache,
-                           rows, scale, window, keep_first, keep_pages, (const float*)gate, gate_stride, gate_col, gate_mode);
+                           v_pitch, rows, scale, window, keep_first, keep_pages, (const float*)gate, gate_stride, gate_col, gate_mode);
   return (int)launch_pdl(wide ? sink_attention_kernel<bf16, WIDE_V_PER_LANE> : sink_attention_kernel<bf16, MAX_V_PER_LANE>,
                          dim3((unsigned)blocks), dim3(warps * 32), smem, stream, (bf16*)out,
                          out_stride, out_col, out_scale, (const bf16*)proj, stride, q_col, HQ, HKV, D, DV, sink, row_seq,
-                         row_pos, seq_slot, table, width, (const bf16*)k_cache, (const bf16*)v_cache, rows, scale, window,
+                         row_pos, seq_slot, table, width, (const bf16*)k_cache, (const bf16*)v_cache, v_pitch, rows, scale, window,
                          keep_first, keep_pages, (const bf16*)gate, gate_stride, gate_col, gate_mode);
 }
 
@@ -594,7 +595,7 @@ KRK_API int krk_sink_attention(void* out, int out_stride, int out_col, float out
 KRK_API int krk_sink_attention_single(void* out, int out_stride, int out_col, float out_scale, const void* proj, int stride,
                                       int q_col, int HQ, int HKV, int D, int DV, const float* sink, const int* seq_slot,
                                       const int* seq_start, const int* table, int width, const void* k_cache,
-                                      const void* v_cache, int n_seqs, float scale, int window, int splits,
+                                      const void* v_cache, int v_pitch, int n_seqs, float scale, int window, int splits,
                                       float* scratch, int fuse, int k_col, int v_col, const float* inv_freq, int rot,
                                       int value_norm, float eps, int keep_first, int keep_pages, const void* gate,
                                       int gate_stride, int gate_col, int gate_mode, int dtype, cudaStream_t stream) {
@@ -605,7 +606,7 @@ KRK_API int krk_sink_attention_single(void* out, int out_stride, int out_col, fl
   if (SPL > 8) return -2;  // the merge kernel holds one factor per block of an item
   const bool wide = DV > 32 * (MAX_V_PER_LANE / 2);  // value rows beyond 128 elements: fewer heads a block
   const int gm = wide ? 4 : GROUP_MAX;
-  if (fuse && (wide || G > GROUP_MAX)) return -2;  // the new key and value are made by one launch per item
+  if (fuse && (wide || G > GROUP_MAX || v_pitch != DV)) return -2;  // the new key and value are made by one launch per item
   if (fuse && (rot < 0 || rot > D || (rot & 1))) return -2;
   {
     const int GN = min(gm, G);  // the most heads a block serves; blocks of the last group may serve fewer
@@ -615,7 +616,7 @@ KRK_API int krk_sink_attention_single(void* out, int out_stride, int out_col, fl
                         (((size_t)D + 7) / 8 * 8 + DV + 8) * esz;
     if (smem > 96 * 1024) return -2;
     cudaError_t e;
-    const bool v4 = (DV & 3) == 0;  // rows of the value cache then start on 8-byte (16 for float) boundaries
+    const bool v4 = (DV & 3) == 0 && (v_pitch & 3) == 0;  // rows of the value cache then start on 8-byte (16 for float) boundaries
     if (dtype == KRK_DTYPE_F32) {
       auto kern = wide ? (v4 ? sink_attention_single_kernel<float, true, false, 16, 4> : sink_attention_single_kernel<float, false, false, 16, 4>)
                   : fuse ? (v4 ? sink_attention_single_kernel<float, true, true, 4, GROUP_MAX> : sink_attention_single_kernel<float, false, true, 4, GROUP_MAX>)
@@ -623,7 +624,7 @@ KRK_API int krk_sink_attention_single(void* out, int out_stride, int out_col, fl
       if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
       e = launch_pdl(kern, dim3(n_seqs * HKV * SPL, groups), dim3(SINGLE_WARPS * 32), smem, stream,
                      (float*)out, out_stride, out_col, out_scale, (const float*)proj, stride, q_col, HQ, HKV, D, DV, sink,
-                     seq_slot, seq_start, table, width, (const float*)k_cache, (const float*)v_cache, scale, window, SPL, scratch, k_col, v_col,
+                     seq_slot, seq_start, table, width, (const float*)k_cache, (const float*)v_cache, v_pitch, scale, window, SPL, scratch, k_col, v_col,
                      inv_freq, rot, value_norm, eps, (float*)k_cache, (float*)v_cache, keep_first, keep_pages,
                      (const float*)gate, gate_stride, gate_col, gate_mode);
     } else {
@@ -633,7 +634,7 @@ KRK_API int krk_sink_attention_single(void* out, int out_stride, int out_col, fl
       if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
       e = launch_pdl(kern, dim3(n_seqs * HKV * SPL, groups), dim3(SINGLE_WARPS * 32), smem, stream,
                      (bf16*)out, out_stride, out_col, out_scale, (const bf16*)proj, stride, q_col, HQ, HKV, D, DV, sink,
-                     seq_slot, seq_start, table, width, (const bf16*)k_cache, (const bf16*)v_cache, scale, window, SPL, scratch, k_col, v_col,
+                     seq_slot, seq_start, table, width, (const bf16*)k_cache, (const bf16*)v_cache, v_pitch, scale, window, SPL, scratch, k_col, v_col,
                      inv_freq, rot, value_norm, eps, (bf16*)k_cache, (bf16*)v_cache, keep_first, keep_pages,
                      (const bf16*)gate, gate_stride, gate_col, gate_mode);
     }

@@ -7,6 +7,9 @@
 // (offset + w), rounded once to the element type T of the path; a second gain gives a
 // second result from the same pass. The gains are float32. One block per row, the row
 // held in shared memory, global memory read once.
+//
+// krk_tanh_norm stands in a norm's place without being one: s = x + f * branch with an optional vector f (float32),
+// y = tanh(alpha * s) * w + b, element by element.
 #include "common.cuh"
 
 namespace {
@@ -116,6 +119,41 @@ __global__ void rmsnorm_wide_kernel(T* __restrict__ out, float* x_new, const flo
   }
 }
 
+// V elements a thread (four where sizes and addresses allow); blockIdx.y walks the row
+template <typename T, bool VEC>
+__global__ void tanh_norm_kernel(T* __restrict__ out, float* x_new, const float* x, const T* __restrict__ branch,
+                                 const float* __restrict__ fold, float alpha, const float* __restrict__ gain,
+                                 const float* __restrict__ shift, int H) {
+  constexpr int V = VEC ? 4 : 1;
+  grid_launch_dependents();
+  const int i = V * (blockIdx.y * blockDim.x + threadIdx.x);
+  if (i >= H) return;
+  const size_t at = (size_t)blockIdx.x * H + i;
+  if (VEC) {
+    const float4 g = *reinterpret_cast<const float4*>(gain + i), h = *reinterpret_cast<const float4*>(shift + i);
+    const float4 c = fold ? *reinterpret_cast<const float4*>(fold + i) : make_float4(1.f, 1.f, 1.f, 1.f);
+    grid_dependency_wait();
+    float4 f = *reinterpret_cast<const float4*>(x + at);
+    if (branch) {
+      float b[4];
+      load4_rows<T>(branch + at, b);
+      f.x += c.x * b[0]; f.y += c.y * b[1]; f.z += c.z * b[2]; f.w += c.w * b[3];
+      *reinterpret_cast<float4*>(x_new + at) = f;
+    }
+    const float r[4] = {tanhf(alpha * f.x) * g.x + h.x, tanhf(alpha * f.y) * g.y + h.y, tanhf(alpha * f.z) * g.z + h.z,
+                        tanhf(alpha * f.w) * g.w + h.w};
+    store4_rows<T>(out + at, r);
+    return;
+  }
+  grid_dependency_wait();
+  float f = x[at];
+  if (branch) {
+    f += (fold ? fold[i] : 1.f) * to_float<T>(branch[at]);
+    x_new[at] = f;
+  }
+  out[at] = from_float<T>(tanhf(alpha * f) * gain[i] + shift[i]);
+}
+
 __device__ __forceinline__ float activation(float z, int act) {
   if (act == 0) return z / (1.0f + expf(-z));                                                   // silu
   if (act == 1) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));  // gelu, tanh form
@@ -193,6 +231,24 @@ KRK_API int krk_rmsnorm_wide(void* out, float* x_new, const float* x, const void
   return dtype == KRK_DTYPE_F32
              ? launch_rmsnorm_wide<float>(out, x_new, x, branch, gain, offset, rows, H, eps, branch2, bscale, gain2, out2, stream)
              : launch_rmsnorm_wide<bf16>(out, x_new, x, branch, gain, offset, rows, H, eps, branch2, bscale, gain2, out2, stream);
+}
+
+template <typename T>
+static int launch_tanh_norm(void* out, float* x_new, const float* x, const void* branch, const float* fold, float alpha,
+                            const float* gain, const float* shift, int rows, int H, cudaStream_t stream) {
+  const bool vec = H % 4 == 0 && (((uintptr_t)gain | (uintptr_t)shift | (uintptr_t)fold) & 15) == 0;
+  const int pieces = vec ? H / 4 : H;
+  const int threads = min(256, (pieces + 31) / 32 * 32);
+  auto kern = vec ? tanh_norm_kernel<T, true> : tanh_norm_kernel<T, false>;
+  return (int)launch_pdl(kern, dim3(rows, (pieces + threads - 1) / threads), dim3(threads), 0, stream, (T*)out, x_new, x,
+                         (const T*)branch, fold, alpha, gain, shift, H);
+}
+
+KRK_API int krk_tanh_norm(void* out, float* x_new, const float* x, const void* branch, const float* fold, float alpha,
+                          const float* gain, const float* shift, int rows, int H, int dtype, cudaStream_t stream) {
+  if (rows == 0) return 0;
+  return dtype == KRK_DTYPE_F32 ? launch_tanh_norm<float>(out, x_new, x, branch, fold, alpha, gain, shift, rows, H, stream)
+                                : launch_tanh_norm<bf16>(out, x_new, x, branch, fold, alpha, gain, shift, rows, H, stream);
 }
 
 KRK_API int krk_gated_act(void* out, const void* gu, int gu_stride, int rows, int I, int act, int row_gate_col, int dtype,

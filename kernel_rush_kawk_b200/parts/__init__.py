@@ -15,9 +15,11 @@ from .wide import DenseMLP, GatedMLP, ScaledEmbedding, WideRMSNorm
 from .branches import Branch, ParallelMixer
 from .sink_attention import SinkWindowAttention
 from .recurrent import DeltaRule, TimeMixWKV
-from .latent_attention import LatentAttention
+from .matrix_memory import GatedLinearAttention, MatrixLSTM
+from .latent_attention import LatentAttention, RotatedLatentAttention
 from .moe import RoutedExperts
 from .hyper import HyperRMSNorm
+from .tanh_norm import TanhNorm
 from .ssm import Mamba2
 from .wrappers import NormedSum, TokenShifted
 

@@ -168,7 +168,8 @@ class Stream:
     the next norm computes x + scale * (branch + branch2).
 
     With hyper-connections ``x`` holds several streams side by side and ``fold`` the
-    weights with which the pending output is written back into them (parts/hyper.py)."""
+    weights with which the pending output is written back into them (parts/hyper.py); a
+    norm that scales outputs element by element leaves that vector there (parts/tanh_norm.py)."""
 
     __slots__ = ("x", "branch", "branch2", "scale", "fold")
 

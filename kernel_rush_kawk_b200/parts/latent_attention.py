@@ -25,6 +25,7 @@ What the cache keeps is the same either way.
 from __future__ import annotations
 
 import copy
+import math
 
 import torch
 
@@ -137,4 +138,97 @@ class LatentAttention(Branch):
         return view, KVView(k, v, table, width, self.window, self.heads, self.dim, self.vdim)
 
 
+def scaled_frequencies(dims: int, base: float, scaling: dict | None) -> tuple[torch.Tensor, float]:
+    """float64 frequencies base^(-2i/dims), i < dims/2, and the factor of cosine and sine. With ``scaling`` (YaRN:
+    factor, original, fast, slow) the frequencies that turn fewer than ``slow`` times over ``original`` positions are
+    divided by the factor, those that turn more than ``fast`` times stay, and a ramp joins them."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    f = base ** (-2.0 * i / max(dims, 1))
+    if scaling is None:
+        return f, 1.0
+    index_of = lambda turns: dims * math.log(scaling["original"] / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+    lo = max(math.floor(index_of(scaling["fast"])), 0)
+    hi = min(math.ceil(index_of(scaling["slow"])), dims - 1)
+    ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+    return f / scaling["factor"] * ramp + f * (1.0 - ramp), 0.1 * math.log(scaling["factor"]) + 1.0
+
+
+class RotatedLatentAttention(Branch):
+    """Latent attention with a rotated part, low-rank queries and a gate per element.
+
+    q = Wuq norm(Wdq h), per head [``dim`` plain, ``rot_dim`` rotated]; Wdkv h is a row of ``kv_rank`` elements, RMS
+    normed into c, and ``rot_dim`` more, rotated: one key part that all heads share. A position leaves [c, rotated part] in
+    the cache. Per head k = Wuk_h c, v = Wuv_h c, score = (q_plain . k + q_rot . k_rot) * scale, causal softmax; the heads
+    side by side are multiplied by sigmoid(Wg h) and projected. Neighbours (2i, 2i + 1) are rotated together.
+
+    A mixer built with ``own_cache`` False has no Wdkv: the rows that it reads were left by another layer's run (the
+    schedule's ``cache_from``); everything else is its own.
+
+    params: hidden, heads, dim, rot_dim, vdim, kv_rank, q_rank, scale, rot_base, rot_scaling (None or factor, original,
+    fast, slow), own_cache (default True), eps."""
+
+    def __init__(self, params):
+        super().__init__(params)
+        p = params
+        self.hidden = int(p["hidden"])
+        self.heads = int(p["heads"])
+        self.dim = int(p["dim"])
+        self.rot = int(p["rot_dim"])
+        self.vdim = int(p["vdim"])
+        self.rank = int(p["kv_rank"])
+        self.q_rank = int(p["q_rank"])
+        self.scale = float(p["scale"])
+        self.rot_base = float(p["rot_base"])
+        self.rot_scaling = None if p.get("rot_scaling") is None else dict(p["rot_scaling"])
+        self.own_cache = bool(p.get("own_cache", True))
+        self.eps = float(p["eps"])
+        if self.rot % 2:
+            raise ValueError(f"rot_dim ({self.rot}) must be even")
+
+    def tensor_specs(self):
+        H, C = self.heads, self.hidden
+        specs = {"dq": TensorSpec((self.q_rank, C)), "dq.norm": TensorSpec((self.q_rank,), "gain"),
+                 "uq": TensorSpec((H * (self.dim + self.rot), self.q_rank)),
+                 "uk": TensorSpec((H * self.dim, self.rank)), "uv": TensorSpec((H * self.vdim, self.rank)),
+                 "g": TensorSpec((H * self.vdim, C)), "o": TensorSpec((C, H * self.vdim))}
+        if self.own_cache:
+            specs.update({"dkv": TensorSpec((self.rank + self.rot, C)), "dkv.norm": TensorSpec((self.rank,), "gain")})
+        return specs
+
+    def cache_need(self):
+        return KVNeed(1, self.rank + self.rot, None, values=False)
+
+    def bind(self, tensors, runtime):
+        self.w = {k: tensors[k] for k in ("dq", "g", "o") + (("dkv",) if self.own_cache else ())}
+        f = lambda key: tensors[key].float().contiguous()
+        self.q_gain = f("dq.norm")
+        self.row_gain = f("dkv.norm") if self.own_cache else None
+        self.w_uq = tensors["uq"].contiguous()
+        # per head: Wuk_h^T [kv_rank, dim] carries a query in, Wuv_h [vdim, kv_rank] carries a result out
+        self.uk_t = tensors["uk"].view(self.heads, self.dim, self.rank).transpose(1, 2).contiguous()
+        self.uv = tensors["uv"].view(self.heads, self.vdim, self.rank).contiguous()
+        self.w_expand = torch.cat([tensors["uk"], tensors["uv"]], dim=0).contiguous()  # [heads * (dim + vdim), kv_rank]
+        freq, self.rot_factor = scaled_frequencies(self.rot, self.rot_base, self.rot_scaling)
+        hi = freq.to(torch.float32)  # two floats each: the float32 value, then what it leaves of the float64 value
+        self.inv_freq = torch.cat([hi, (freq - hi.double()).to(torch.float32)]).contiguous().to(runtime.device)
+        self.bind_standalone()
+
+    def in_weight(self):
+        # the parts that kernels read in 16-byte pieces come first; any column may follow
+        return torch.cat([self.w["dq"], self.w["g"]] + ([self.w["dkv"]] if self.own_cache else []), dim=0)
+
+    def out_weight(self):
+        return self.w["o"]
+
+    def middle(self, ctx, proj, cache, out, col0, scale):
+        ops = ctx.ops
+        g_col = self.q_rank
+        rows = (g_col + self.heads * self.vdim, self.rank, self.row_gain) if self.own_cache else None
+        cq = ops.latent_rows(proj, (0, self.q_rank, self.q_gain), rows, self.rot, self.inv_freq, self.rot_factor, self.eps,
+                             ctx.batch, cache)
+        q = ops.linear(cq, self.w_uq)
+        ops.rotated_latent_attention(q, self, ctx.batch, cache, (proj, g_col), out, col0, scale, ctx.shared)
+
+
 register_mixer("latent_attention", LatentAttention)
+register_mixer("rotated_latent_attention", RotatedLatentAttention)

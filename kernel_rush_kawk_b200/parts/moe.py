@@ -13,6 +13,13 @@ equal groups of neighbours; a group's score is the sum of its two largest choice
 has one expert), only the ``keep_groups`` best groups' experts can be chosen, and the weights are the chosen
 experts' s divided by their sum (+ 1e-20) and multiplied by ``route_scale``.
 
+"softmax_groups" chooses and weighs by the softmax over all outputs of the router: s = softmax(z), the choice by
+s + correction, a group's score its largest choice score, the weights the chosen s as they are. There the last
+``identity`` of the router's experts + identity outputs are experts without tensors that hand their input through:
+chosen, they add weight * h. Groups are formed over experts and identity experts together.
+
+Without ``gated`` an expert is Wdown_e act(Wup_e h), and so is the shared expert.
+
 The routing never leaves the device: a routing kernel writes each row's experts and
 weights; few rows (single-token steps) read each chosen expert's weights once per
 (row, expert) pair; many rows are counted, ordered by expert and multiplied by all
@@ -34,8 +41,9 @@ class RoutedExperts(FeedForward):
     """params: hidden, experts, top, intermediate, activation ("silu"), shared_intermediate (None or int),
     shared_gate (bool: the shared expert sits behind sigmoid(Wsg h)), router_bias (default True: the router
     has a bias "router.b"), weights ("chosen", the default: softmax over the chosen logits; "all": each chosen
-    expert's share of the softmax over all experts, not renormalised), scoring (None or "sigmoid_groups", with
-    groups, keep_groups and route_scale; it has the tensor "correction" and no router bias)."""
+    expert's share of the softmax over all experts, not renormalised), scoring (None, "sigmoid_groups" with
+    groups, keep_groups and route_scale, or "softmax_groups" with groups, keep_groups and identity; both have the tensor
+    "correction" and no router bias), gated (default True: experts have a gate product)."""
 
     def __init__(self, params):
         super().__init__(params)
@@ -50,37 +58,44 @@ class RoutedExperts(FeedForward):
         self.router_bias = bool(p.get("router_bias", True))
         self.weights = str(p.get("weights", "chosen"))
         self.scoring = p.get("scoring")
-        if self.scoring not in (None, "sigmoid_groups"):
-            raise ValueError(f"scoring must be None or 'sigmoid_groups', got {self.scoring!r}")
+        if self.scoring not in (None, "sigmoid_groups", "softmax_groups"):
+            raise ValueError(f"scoring must be None, 'sigmoid_groups' or 'softmax_groups', got {self.scoring!r}")
+        self.gated = bool(p.get("gated", True))
+        self.identity = int(p.get("identity", 0))
+        if self.identity and self.scoring != "softmax_groups":
+            raise ValueError("identity experts come with 'softmax_groups' scoring")
+        outputs = self.outputs = self.experts + self.identity
         self.groups = int(p.get("groups", 1))
         self.keep_groups = int(p.get("keep_groups", self.groups))
         self.route_scale = float(p.get("route_scale", 1.0))
         if self.scoring:
             self.router_bias = False
-            if self.experts % self.groups or not 1 <= self.keep_groups <= self.groups:
-                raise ValueError(f"{self.experts} experts do not form {self.groups} equal groups of which {self.keep_groups} are kept")
-            if self.top > self.keep_groups * (self.experts // self.groups):
+            if outputs % self.groups or not 1 <= self.keep_groups <= self.groups:
+                raise ValueError(f"{outputs} experts do not form {self.groups} equal groups of which {self.keep_groups} are kept")
+            if self.top > self.keep_groups * (outputs // self.groups):
                 raise ValueError("a token cannot take more experts than the kept groups hold")
         if self.weights not in ("chosen", "all"):
             raise ValueError(f"weights must be 'chosen' or 'all', got {self.weights!r}")
-        if not 1 <= self.top <= self.experts:
-            raise ValueError(f"a token takes between 1 and {self.experts} experts, got top = {self.top}")
+        if not 1 <= self.top <= outputs:
+            raise ValueError(f"a token takes between 1 and {outputs} experts, got top = {self.top}")
         if self.top > 32:
             raise ValueError("at most 32 experts per token")
 
     def tensor_specs(self):
         H, F = self.hidden, self.intermediate
-        specs = {"router": TensorSpec((self.experts, H))}
+        specs = {"router": TensorSpec((self.outputs, H))}
         if self.router_bias:
             specs["router.b"] = TensorSpec((self.experts,), "vector")
         if self.scoring:
-            specs["correction"] = TensorSpec((self.experts,), "vector")
+            specs["correction"] = TensorSpec((self.outputs,), "vector")
         for e in range(self.experts):
-            specs[f"e{e}.gate"] = TensorSpec((F, H))
+            if self.gated:
+                specs[f"e{e}.gate"] = TensorSpec((F, H))
             specs[f"e{e}.up"] = TensorSpec((F, H))
             specs[f"e{e}.down"] = TensorSpec((H, F))
         if self.shared is not None:
-            specs["shared.gate"] = TensorSpec((self.shared, H))
+            if self.gated:
+                specs["shared.gate"] = TensorSpec((self.shared, H))
             specs["shared.up"] = TensorSpec((self.shared, H))
             specs["shared.down"] = TensorSpec((H, self.shared))
             if self.shared_gate:
@@ -93,11 +108,12 @@ class RoutedExperts(FeedForward):
         self.router_w = torch.cat([tensors["router"]] + ([tensors["shared.sg"]] if self.shared_gate else []), dim=0).contiguous()
         self.router_b = tensors["router.b"].float().contiguous() if self.router_bias else None
         self.correction = tensors["correction"].float().contiguous() if self.scoring else None
-        self.w_gate_up = torch.stack([torch.cat([tensors[f"e{e}.gate"], tensors[f"e{e}.up"]], dim=0) for e in range(E)]).contiguous()
+        first = ("gate", "up") if self.gated else ("up",)  # what is stacked into an expert's first product
+        self.w_gate_up = torch.stack([torch.cat([tensors[f"e{e}.{k}"] for k in first], dim=0) for e in range(E)]).contiguous()
         self.w_down = torch.stack([tensors[f"e{e}.down"] for e in range(E)]).contiguous()
         self.w_shared_in = self.w_shared_down = None
         if self.shared is not None:
-            self.w_shared_in = torch.cat([tensors["shared.gate"], tensors["shared.up"]], dim=0).contiguous()
+            self.w_shared_in = torch.cat([tensors["shared." + k] for k in first], dim=0).contiguous()
             self.w_shared_down = tensors["shared.down"].contiguous()
 
     def forward(self, ctx, h):
@@ -105,7 +121,15 @@ class RoutedExperts(FeedForward):
         x = h.tensor() if hasattr(h, "tensor") and not isinstance(h, torch.Tensor) else h
         base = None
         if self.shared is not None:
-            base = ops.linear(ops.gate_up_act(x, self.w_shared_in, self.shared, self.activation), self.w_shared_down)
+            act = (ops.gate_up_act(x, self.w_shared_in, self.shared, self.activation) if self.gated
+                   else ops.up_act(x, self.w_shared_in, self.activation))
+            base = ops.linear(act, self.w_shared_down)
+        if self.scoring == "softmax_groups":
+            experts, weights, row_gate, passed = ops.moe_route_softmax_groups(x, self.router_w, self.correction, self.top,
+                                                                              self.groups, self.keep_groups, self.identity,
+                                                                              gate_row=self.shared_gate)
+            return ops.moe_experts(x, self.w_gate_up, self.w_down, experts, weights, self.intermediate, self.activation,
+                                   add=base, add_gate=row_gate, batch=ctx.batch, gated=self.gated, add_input=passed)
         if self.scoring:
             experts, weights, row_gate = ops.moe_route(x, self.router_w, None, self.top, gate_row=self.shared_gate,
                                                        sigmoid_groups=(self.correction, self.groups, self.keep_groups,
@@ -116,7 +140,7 @@ class RoutedExperts(FeedForward):
         else:
             experts, weights, row_gate = ops.moe_route(x, self.router_w, self.router_b, self.top, gate_row=self.shared_gate)
         return ops.moe_experts(x, self.w_gate_up, self.w_down, experts, weights, self.intermediate, self.activation,
-                               add=base, add_gate=row_gate, batch=ctx.batch)
+                               add=base, add_gate=row_gate, batch=ctx.batch, **({} if self.gated else {"gated": False}))
 
 
 register_feed_forward("routed_experts", RoutedExperts)
