@@ -175,6 +175,8 @@ def _act(z, name):
         return z * torch.sigmoid(z)
     if name == "sigmoid":
         return torch.sigmoid(z)
+    if name == "relu2":
+        return torch.clamp(z, min=0.0) ** 2
     if name == "gelu_tanh":
         return 0.5 * z * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (z + 0.044715 * z ** 3)))
     raise ValueError(name)
@@ -427,17 +429,22 @@ class _WideOps:
         out[:, out_col:out_col + inner] = (v.reshape(rows, inner) * weight * out_scale).to(out.dtype)
 
     def moe_experts(self, x, w_gate_up, w_down, experts, weights, intermediate, activation, add=None, add_gate=None,
-                    batch=None):
+                    batch=None, gated=True, add_input=None):
         rows, top = experts.shape
         out = torch.zeros((rows, w_down.shape[1]), dtype=torch.float32) if add is None else add.float().clone()
         if add is not None and add_gate is not None:
             out = out * add_gate[:, None]
         xf = x.float()
+        if add_input is not None:
+            out = out + add_input[:, None] * xf
         for r in range(rows):
             for j in range(top):
                 e = int(experts[r, j])
+                if e < 0:
+                    continue
                 gu = xf[r] @ w_gate_up[e].float().t()
-                a = (_act(gu[:intermediate], activation) * gu[intermediate:]).to(self.dtype).float()
+                a = _act(gu[:intermediate], activation)
+                a = (a * gu[intermediate:] if gated else a).to(self.dtype).float()
                 out[r] += weights[r, j] * (a @ w_down[e].float().t())
         return out.to(self.dtype)
 
@@ -564,6 +571,121 @@ class _WideOps:
         o = o * torch.rsqrt((o * o).mean(dim=-1, keepdim=True) + eps)
         res = o.reshape(rows, H * N) * norm_w.float() * g * out_scale
         out[:, out_col:out_col + H * N] = res.to(out.dtype)
+
+    # -- tanh in a norm's place, matrix states without a removal term, latent attention with a rotated part, softmax
+    # routing within groups with identity experts -----------------------------------------------------------------
+    def tanh_norm(self, x, branch, fold, alpha, gain, shift, x_new, out_dtype):
+        s = x
+        if branch is not None:
+            s = x + (branch.float() if fold is None else fold * branch.float())
+            x_new.copy_(s)
+        return (torch.tanh(alpha * s) * gain + shift).to(out_dtype)
+
+    def _memory(self, q, k, v, gates_of, heads, dim, vdim, batch, state, nm=None):
+        """gates_of(row) -> (decay of the state's rows, factor of k v^T, new running maximum or None)"""
+        rows = q.shape[0]
+        qq, kk = q.float().reshape(rows, heads, dim) * dim ** -0.5, k.float().reshape(rows, heads, dim)
+        vv = v.float().reshape(rows, heads, vdim)
+        o = torch.empty((rows, heads, vdim), dtype=torch.float32)
+        row0 = 0
+        for slot, n in zip(batch.slots, batch.q_lens):
+            S = state[slot].clone()
+            nv = None if nm is None else nm[slot, :, :dim].clone()
+            m = None if nm is None else nm[slot, :, dim].clone()
+            for t in range(row0, row0 + n):
+                keep, take, m = gates_of(t, m)
+                S = keep * S + take * kk[t][:, :, None] * vv[t][:, None, :]
+                o[t] = torch.einsum("hnp,hn->hp", S, qq[t])
+                if nm is not None:
+                    nv = keep[..., 0] * nv + take[..., 0] * kk[t]
+                    o[t] /= torch.maximum((nv * qq[t]).sum(-1).abs(), torch.exp(-m))[:, None] + 1e-6
+            state[slot] = S
+            if nm is not None:
+                nm[slot, :, :dim], nm[slot, :, dim] = nv, m
+            row0 += n
+        return o
+
+    def gla_scan(self, q, k, v, gate, lora, w2, bias, tau, heads, dim, vdim, norm_w, eps, state, batch, out, out_col, out_scale):
+        rows = q.shape[0]
+        z = lora.float() @ w2.float().t() + bias
+        alpha = torch.exp(torch.nn.functional.logsigmoid(z) / tau).reshape(rows, heads, dim, 1)
+        o = self._memory(q, k, v, lambda t, m: (alpha[t], 1.0, None), heads, dim, vdim, batch, state)
+        o = o * torch.rsqrt((o * o).mean(dim=-1, keepdim=True) + eps) * norm_w
+        g = gate.float()
+        out[:, out_col:out_col + heads * vdim] = (o.reshape(rows, -1) * g * torch.sigmoid(g) * out_scale).to(out.dtype)
+
+    def mlstm_scan(self, q, k, v, gate, if_rows, if_bias, cap, heads, dim, vdim, norm_w, eps, state, nm, batch, out, out_col,
+                   out_scale):
+        rows = q.shape[0]
+        z = cap * torch.tanh((if_rows.float() + if_bias) / cap)
+        i, f = z[:, :heads], torch.nn.functional.logsigmoid(z[:, heads:])
+
+        def gates_of(t, m):
+            m_new = torch.maximum(f[t] + m, i[t])
+            return torch.exp(f[t] + m - m_new)[:, None, None], torch.exp(i[t] - m_new)[:, None, None], m_new
+
+        o = self._memory(q, k, v, gates_of, heads, dim, vdim, batch, state, nm)
+        o = (o * torch.rsqrt((o * o).mean(dim=-1, keepdim=True) + eps)).reshape(rows, -1)
+        out[:, out_col:out_col + heads * vdim] = (o * norm_w * torch.sigmoid(gate.float()) * out_scale).to(out.dtype)
+
+    @staticmethod
+    def _turn_pairs(x, pos, inv_freq, factor):
+        half = x.shape[-1] // 2
+        a = pos.double()[:, None] * (inv_freq[:half].double() + inv_freq[half:].double())[None, :]
+        c, s = (torch.cos(a) * factor).float(), (torch.sin(a) * factor).float()
+        while c.dim() < x.dim():
+            c, s = c.unsqueeze(1), s.unsqueeze(1)
+        u, v = x[..., 0::2].float(), x[..., 1::2].float()
+        return torch.stack([u * c - v * s, v * c + u * s], dim=-1).reshape(x.shape)
+
+    def latent_rows(self, proj, query, rows, rot_dim, inv_freq, rot_factor, eps, batch, cache):
+        col, n, gain = query
+        norm = lambda x, g: (x * torch.rsqrt((x * x).mean(dim=-1, keepdim=True) + eps) * g).to(proj.dtype)
+        if rows is not None:
+            c_col, rank, c_gain = rows
+            pos = batch.row_pos.long()
+            page = cache.table.long()[batch.seq_slot.long()[batch.row_seq.long()], (pos // PAGE) % cache.width]
+            cache.k[page, 0, pos % PAGE, :rank] = norm(proj[:, c_col:c_col + rank].float(), c_gain)
+            cache.k[page, 0, pos % PAGE, rank:] = self._turn_pairs(proj[:, c_col + rank:c_col + rank + rot_dim], pos, inv_freq,
+                                                                   rot_factor).to(proj.dtype)
+        return norm(proj[:, col:col + n].float(), gain)
+
+    def rotated_latent_attention(self, q, m, batch, cache, gate, out, out_col, out_scale, shared):
+        rows, H, D, P, R = q.shape[0], m.heads, m.dim, m.vdim, m.rank
+        q = q.reshape(rows, H, D + m.rot)
+        qr = self._turn_pairs(q[..., D:], batch.row_pos.long(), m.inv_freq, m.rot_factor).to(q.dtype)
+        g = torch.sigmoid(gate[0][:, gate[1]:gate[1] + H * P].float())
+        res = torch.empty((rows, H, P), dtype=torch.float32)
+        row0 = 0
+        for slot, start, n in zip(batch.slots, batch.starts, batch.q_lens):
+            positions = torch.arange(start + n)
+            row = cache.k[cache.table.long()[slot, (positions // PAGE) % cache.width], 0, positions % PAGE].float()
+            k = torch.einsum("jr,hrd->jhd", row[:, :R], m.uk_t.float())
+            v = torch.einsum("jr,hpr->jhp", row[:, :R], m.uv.float())
+            s = (torch.einsum("ihd,jhd->hij", q[row0:row0 + n, :, :D].float(), k)
+                 + torch.einsum("ihd,jd->hij", qr[row0:row0 + n].float(), row[:, R:])) * m.scale
+            s = s.masked_fill(positions[None, None, :] > torch.arange(start, start + n)[None, :, None], float("-inf"))
+            res[row0:row0 + n] = torch.einsum("hij,jhp->ihp", torch.softmax(s, dim=-1), v)
+            row0 += n
+        out[:, out_col:out_col + H * P] = (res.reshape(rows, H * P) * g * out_scale).to(out.dtype)
+
+    def moe_route_softmax_groups(self, x, w, correction, top, groups, keep, identity, gate_row=False):
+        z = x.float() @ w.float().t()
+        row_gate = torch.sigmoid(z[:, -1]) if gate_row else None
+        z = z[:, :-1] if gate_row else z
+        rows, n = z.shape
+        s = torch.softmax(z, dim=-1)
+        c = s + correction
+        best = c.view(rows, groups, n // groups).max(dim=-1).values.topk(keep, dim=-1).indices
+        allowed = torch.zeros((rows, groups), dtype=torch.bool, device=c.device).scatter_(1, best, True)
+        idx = c.masked_fill(~allowed.repeat_interleave(n // groups, dim=1), float("-inf")).topk(top, dim=-1).indices
+        wt = s.gather(1, idx)
+        handed = idx >= n - identity
+        passed = (wt * handed).sum(-1) if identity else None
+        return torch.where(handed, -1, idx).to(torch.int32), wt * ~handed, row_gate, passed
+
+    def up_act(self, h, w_up, activation):
+        return self.act_rows(self.linear(h, w_up), activation)
 
 
 for _name, _fn in vars(_WideOps).items():
