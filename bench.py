@@ -43,6 +43,13 @@ and routed feed-forwards chosen by sigmoid scores within groups) at two sizes be
 the Taredra hybrid decoder of equal width, feed-forward, heads and layer count, and beside the Qwen3 decoder of
 that size.
 
+``--only design_zefapel`` measures the Zefapel decoder (matrix memories with exponential gates, gated linear attention,
+latent attention with a rotated part whose rows two layers share, dense and routed feed-forwards with identity experts
+and a shared one, tanh in the norms' place) at two sizes beside its closest existing model, the Disorax decoder of equal
+width and heads (attention over cached low-rank rows, routed experts with a shared one, a 32-bit stream), beside the
+Zadunex decoder of about that size (the other model whose matrix states outweigh its attention), and beside the Qwen3
+decoder of that size.
+
 ``--only workload_8b`` and ``--only workload_14b`` run the baseline's two larger
 configurations (Qwen3-8B sizes: 8 prompts of 256 to 2,048 tokens, 128 greedy steps;
 Qwen3-14B sizes: 16 prompts of 512 to 4,096 tokens, 128 steps at temperature 0.7)
@@ -222,24 +229,30 @@ DESIGN_SIZES = {
                    "head_dim": 128, "vocab_size": 32768},
     "zadunex_4b": {"hidden_size": 2560, "intermediate_size": 9728, "num_attention_heads": 32, "num_key_value_heads": 8,
                    "head_dim": 128, "vocab_size": 32768},
+    "zefapel_small": {"hidden_size": 1024, "intermediate_size": 3072, "num_attention_heads": 8, "num_key_value_heads": 2,
+                      "head_dim": 128, "vocab_size": 32768},
+    "zefapel_lite": {"hidden_size": 2048, "intermediate_size": 8192, "num_attention_heads": 16, "num_key_value_heads": 4,
+                     "head_dim": 128, "vocab_size": 32768},
     "fogizen_1b": {"hidden_size": 1536, "intermediate_size": 6144, "num_attention_heads": 12, "num_key_value_heads": 4,
                    "head_dim": 128, "vocab_size": 32768},
     "fogizen_4b": {"hidden_size": 2560, "intermediate_size": 9728, "num_attention_heads": 32, "num_key_value_heads": 8,
                    "head_dim": 128, "vocab_size": 151936},
 }
-#: a design's closest existing model of equal size, measured beside it as well (preset -> preset)
-DESIGN_NEIGHBOURS = {"zadunex_1b": "taredra_1b", "zadunex_4b": "taredra_4b", "fogizen_1b": "taredra_1b",
-                     "fogizen_4b": "taredra_4b"}
+#: a design's closest existing model of equal size, measured beside it as well (preset -> presets)
+DESIGN_NEIGHBOURS = {"zadunex_1b": ("taredra_1b",), "zadunex_4b": ("taredra_4b",), "fogizen_1b": ("taredra_1b",),
+                     "fogizen_4b": ("taredra_4b",), "zefapel_small": ("disorax_small", "zadunex_1b"),
+                     "zefapel_lite": ("disorax_lite", "zadunex_4b")}
 KERNEL_FAMILIES = {
     "product": ("_skinny", "_library_gemm", "_gemm_nt", "gemm_tcgen05"),
-    "norm": ("rmsnorm", "add_rmsnorm", "rmsnorm_wide", "hyper_rmsnorm", "norm_sum"),
+    "norm": ("rmsnorm", "add_rmsnorm", "rmsnorm_wide", "hyper_rmsnorm", "norm_sum", "tanh_norm"),
     "activation": ("swiglu", "gated_act", "act_rows"),
     "attention": ("rope_attention", "rotate_norm_write", "sink_attention", "latent_norm_write", "head_linear",
-                  "bias_row_norm", "bias_norm_rotate_write", "mixed_attention"),
-    "recurrence": ("token_shift", "linear_recurrence", "causal_conv_silu", "ssd_scan", "gated_group_norm"),
+                  "bias_row_norm", "bias_norm_rotate_write", "mixed_attention", "latent_rows", "rotated_latent_attention"),
+    "recurrence": ("token_shift", "linear_recurrence", "causal_conv_silu", "ssd_scan", "gated_group_norm", "gla_scan",
+                   "mlstm_scan"),
     # routing and the routed experts; for steps of many tokens this holds the experts' dense products too, which
     # the product family counts as well
-    "experts": ("moe_route", "moe_experts"),
+    "experts": ("moe_route", "moe_route_softmax_groups", "moe_experts"),
     "embedding": ("embed", "embed_scaled", "embed_bigram", "gather_rows"),
 }
 
@@ -350,10 +363,10 @@ def run_designs(args) -> dict:
         q_cfg = Qwen3Config.from_dict({**twin, "num_hidden_layers": layers, "rms_norm_eps": 1e-6, "rope_theta": 1e4,
                                        "tie_word_embeddings": True, "max_position_embeddings": CONTEXT})
         out["sizes"][preset] = {"layers": layers, design: measure(t_cfg, t_cfg.vocab)}
-        if preset in DESIGN_NEIGHBOURS:
-            n_cfg = preset_config(DESIGN_NEIGHBOURS[preset])
+        for neighbour in DESIGN_NEIGHBOURS.get(preset, ()):
+            n_cfg = preset_config(neighbour)
             n_cfg = type(n_cfg).from_dict({**n_cfg.to_dict(), "layers": n_cfg.to_dict()["layers"][:layers]})
-            out["sizes"][preset][DESIGN_NEIGHBOURS[preset]] = measure(n_cfg, n_cfg.vocab)
+            out["sizes"][preset][neighbour] = measure(n_cfg, n_cfg.vocab)
         out["sizes"][preset]["qwen3"] = measure(q_cfg, q_cfg.vocab_size)
     return out
 
@@ -665,7 +678,7 @@ def main() -> int:
     p.add_argument("--impl", default="ours", choices=["ours", "reference"])
     p.add_argument("--only", default="", choices=["", "prefill", "decode_b1", "decode_b8", "decode_b16", "decode_b32", "decode_b64",
                                                   "workload_8b", "workload_14b", "design_taredra", "design_disorax",
-                                                  "design_zadunex", "design_fogizen"],
+                                                  "design_zadunex", "design_fogizen", "design_zefapel"],
                    help="run one piece only (for profiling), or one of the baseline's larger configurations end to end")
     p.add_argument("--layers", type=int, default=0, help="run fewer layers than the model has (both numbers are reported)")
     args = p.parse_args()

@@ -97,7 +97,15 @@ _MEMORY_SIGNATURES = {
     "krk_memory_decays": [_P, _P, c_int, _P, _P, c_float, c_int, c_int, c_int, c_int, _P],
     "krk_memory_scan": [_P, _P, c_int, _P, c_int, _P, c_int, c_float, _P, _P, _P, _P, c_int, c_int, c_int, c_int, _P, _P, _P,
                         c_int, _P],
+    "krk_memory_chunk_tokens": [c_int, c_int, c_int],
+    "krk_memory_chunk_decays": [_P, _P, c_int, _P, _P, c_float, c_int, c_int, c_int, c_int, _P, _P, _P],
+    "krk_memory_chunks": [_P, _P, c_int, _P, c_int, _P, c_int, c_float, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int,
+                          _P, _P, _P, _P],
     "krk_memory_finish": [_P, c_int, c_int, c_float, _P, _P, _P, c_int, _P, c_int, c_int, c_float, c_int, c_int, _P],
+}
+_LATENT_SIGNATURES = {
+    "krk_latent_prefill": [_P, c_int, c_float, _P, c_int, c_int, c_int, _P, _P, c_int, c_int, _P, c_float, c_float, c_int, c_int,
+                           _P, _P, _P, _P, _P, c_int, _P],
 }
 _SCAN_SIGNATURES = {
     "krk_token_shift": [_P, _P, c_int, _P, _P, c_int, c_int, c_int, _P, _P, _P, c_int, _P, c_int],
@@ -162,6 +170,7 @@ class Kernels:
         self.core = _load(build_library("core"), _SIGNATURES)
         self._mix = self._scan = self._moe = self._memory = None
         self.attn: dict[int, ctypes.CDLL] = {}
+        self.latent: dict[tuple, ctypes.CDLL] = {}
         for d in head_dims:
             self._attn_lib(int(d))
         self.error = torch.zeros(1, dtype=torch.int32, device=self.device)
@@ -193,6 +202,14 @@ class Kernels:
                 raise KernelError(f"attention kernels take an even head size up to 256, got {head_dim}")
             lib = self.attn[head_dim] = _load(build_library("attn", head_dim), _ATTN_SIGNATURES)
             assert lib.krk_attention_head_dim() == head_dim
+        return lib
+
+    def _latent_lib(self, key_dim: int, value_dim: int) -> ctypes.CDLL:
+        """The prompt attention of a pair of head sizes over keys and values made from latent rows, compiled and loaded
+        at its first call."""
+        lib = self.latent.get((key_dim, value_dim))
+        if lib is None:
+            lib = self.latent[(key_dim, value_dim)] = _load(build_library("latent", (key_dim, value_dim)), _LATENT_SIGNATURES)
         return lib
 
     # -- plumbing -------------------------------------------------------------
@@ -688,6 +705,8 @@ class Kernels:
         g_ptr, g_stride = self._rows_view(gate[0])
         g_ptr += int(gate[1]) * gate[0].element_size()
         optr, ostride = self._rows_view(out)
+        if self._latent_prefill(q, m, batch, cache, g_ptr, g_stride, optr, ostride, out_col, out_scale, shared):
+            return
         # a head's query is carried into the latent space, attention runs over the cached rows themselves
         qx = torch.empty((rows, H * W), dtype=q.dtype, device=q.device)
         self._ok(self.mix.krk_head_linear(qx.data_ptr(), H * W, 0, W, 1.0, q.data_ptr(), q.stride(0), D + E, m.uk_t.data_ptr(), H,
@@ -698,6 +717,45 @@ class Kernels:
         self._ok(self.mix.krk_head_linear(optr, ostride, int(out_col), P, float(out_scale), mixed.data_ptr(), H * R, R,
                                           m.uv.data_ptr(), H, P, R, rows, 0, None, 1.0, None, g_ptr, g_stride, _code(q.dtype),
                                           self._stream()), "values out of the latent space")
+
+    LATENT_DENSE_BYTES = 4 << 30  # keys and values of a step's whole context beyond this size are not written out
+
+    def _latent_prefill(self, q, m, batch, cache, g_ptr, g_stride, optr, ostride, out_col, out_scale, shared) -> bool:
+        """A step of many tokens in bfloat16: the sequences' cached rows as one dense matrix, keys and values from it by one
+        product, tensor-core attention over those. False where the step or the sizes are not of that kind."""
+        H, D, E, R, P = m.heads, m.dim, m.rot, m.rank, m.vdim
+        if (batch.is_decode or q.dtype != torch.bfloat16 or D % 8 or E % 8 or R % 8 or (D + E) % 16 or P % 16 or D + E > 256
+                or P > 256 or q.stride(0) % 8):
+            return False
+        lengths = [s + n for s, n in zip(batch.starts, batch.q_lens)]
+        if 2 * sum(lengths) * H * (D + P) > self.LATENT_DENSE_BYTES:
+            return False
+        offsets = shared.get("latent_offsets")
+        if offsets is None:
+            at, first = [], 0
+            for n in lengths:
+                at.append(first)
+                first += n
+            offsets = shared["latent_offsets"] = torch.tensor(at, dtype=torch.int32).to(q.device)
+        key = ("latent_rows", cache.k.data_ptr())  # layers that read one cache share the matrix
+        rows = shared.get(key)
+        if rows is None:
+            rows = shared[key] = torch.empty((sum(lengths), R + E), dtype=q.dtype, device=q.device)
+            self._ok(self.mix.krk_latent_gather(rows.data_ptr(), cache.k.data_ptr(), R + E, batch.n_seqs, max(lengths),
+                                                batch.seq_slot.data_ptr(), batch.seq_start.data_ptr(), batch.seq_qlen.data_ptr(),
+                                                offsets.data_ptr(), cache.table.data_ptr(), cache.width, _code(q.dtype),
+                                                self._stream()), "cached rows as a matrix")
+        latent = rows[:, :R]
+        kv = self.linear(latent if rows.shape[0] > self.SKINNY_MAX_ROWS else latent.contiguous(), m.w_expand)
+        rc = self._latent_lib(D + E, P).krk_latent_prefill(
+            optr + int(out_col) * 2, ostride, float(out_scale), q.data_ptr(), q.stride(0), H, D, kv.data_ptr(), rows.data_ptr(),
+            R + E, R, m.inv_freq.data_ptr(), float(m.rot_factor), float(m.scale), batch.n_seqs, batch.max_q_len,
+            batch.seq_start.data_ptr(), batch.seq_qlen.data_ptr(), batch.cu_q.data_ptr(), offsets.data_ptr(), g_ptr, g_stride,
+            self._stream())
+        if rc == -2:  # odd strides or offsets; the general kernels take them
+            return False
+        self._ok(rc, "prompt attention over latent rows")
+        return True
 
     # -- routed experts ------------------------------------------------------------------------
     MOE_PAIR_ROWS = 16  # rows up to which every (row, expert) pair reads its expert's weights by itself
@@ -1084,46 +1142,78 @@ class Kernels:
         self._ok(rc, f"{kind} recurrence (heads of up to 256 channels)")
 
     # -- matrix states without a removal term -------------------------------------------------
-    def _memory_scan(self, q, k, v, gate, decays, gates, heads, dim, vdim, norm_w, eps, state, nm, batch, out, out_col, out_scale):
-        views = [self._rows_view(t) for t in (q, k, v, gate)]
+    MEMORY_CHUNK_MIN = 128  # tokens of a step's longest sequence from which a bfloat16 scan runs in chunks
+
+    def _memory_chunk(self, views, dtype, dim, vdim, gated, batch) -> int:
+        """Tokens per chunk where a step's scan runs in chunks on the tensor cores, else 0."""
+        if batch.is_decode or dtype != torch.bfloat16 or batch.max_q_len < self.MEMORY_CHUNK_MIN or any(
+                p % 16 or s % 8 for p, s in views[:3]):
+            return 0
+        return int(self.memory.krk_memory_chunk_tokens(dim, vdim, int(gated)))
+
+    def _memory_scan(self, views, chunk, dtype, decays, gates, heads, dim, vdim, norm_w, eps, state, nm, batch, rows, out,
+                     out_col, out_scale):
         optr, ostride = self._rows_view(out)
-        rows = q.shape[0]
         if state.dtype != torch.float32 or not state.is_contiguous() or state.shape[1:] != (heads, dim, vdim):
             raise KernelError("the scan keeps a contiguous float32 state [slots, heads, dim, vdim]")
         if nm is not None and (nm.dtype != torch.float32 or not nm.is_contiguous() or nm.shape[1:] != (heads, dim + 1)):
             raise KernelError("the gated scan keeps a contiguous float32 [slots, heads, dim + 1] beside its state")
-        y = torch.empty((rows, heads * (vdim + int(nm is not None))), dtype=torch.float32, device=q.device)
-        self._ok(self.memory.krk_memory_scan(y.data_ptr(), *views[0], *views[1], *views[2], float(dim) ** -0.5, _ptr(decays),
-                                             _ptr(gates), state.data_ptr(), _ptr(nm), heads, dim, vdim, batch.n_seqs,
-                                             batch.cu_q.data_ptr(), batch.seq_qlen.data_ptr(), batch.seq_slot.data_ptr(),
-                                             _code(q.dtype), self._stream()), "matrix-state scan (up to 1,024 key channels a head)")
+        gated = nm is not None
+        y = torch.empty((rows, heads * (vdim + int(gated))), dtype=torch.float32, device=self.device)
+        tables = (batch.cu_q.data_ptr(), batch.seq_qlen.data_ptr(), batch.seq_slot.data_ptr())
+        if chunk:
+            chunks = batch.n_seqs * -(-batch.max_q_len // chunk) * heads
+            cs = torch.empty((chunks, dim * (vdim + int(gated))), dtype=torch.float32, device=self.device)
+            cd = torch.empty((chunks, dim), dtype=torch.float32, device=self.device)
+            self._ok(self.memory.krk_memory_chunks(y.data_ptr(), *views[0], *views[1], *views[2], float(dim) ** -0.5, _ptr(decays),
+                                                   _ptr(gates), state.data_ptr(), _ptr(nm), cs.data_ptr(), cd.data_ptr(), heads,
+                                                   dim, vdim, batch.n_seqs, batch.max_q_len, *tables, self._stream()),
+                     "matrix-state scan in chunks")
+            self.launches += 2
+        else:
+            self._ok(self.memory.krk_memory_scan(y.data_ptr(), *views[0], *views[1], *views[2], float(dim) ** -0.5, _ptr(decays),
+                                                 _ptr(gates), state.data_ptr(), _ptr(nm), heads, dim, vdim, batch.n_seqs, *tables,
+                                                 _code(dtype), self._stream()),
+                     "matrix-state scan (up to 1,024 key channels a head)")
         self._ok(self.memory.krk_memory_finish(optr, ostride, int(out_col), float(out_scale), y.data_ptr(), _ptr(gates), *views[3],
-                                               norm_w.data_ptr(), heads, vdim, float(eps), rows, _code(q.dtype), self._stream()),
+                                               norm_w.data_ptr(), heads, vdim, float(eps), rows, _code(dtype), self._stream()),
                  "matrix-state head norm and gate")
 
     def gla_scan(self, q, k, v, gate, lora, w2, bias, tau, heads, dim, vdim, norm_w, eps, state, batch, out, out_col, out_scale):
         """Gated linear attention over a step's rows, from and to ``state`` [slots, heads, dim, vdim]; see
         csrc/matrix_memory.cu. ``norm_w`` [vdim]."""
+        views = [self._rows_view(t) for t in (q, k, v, gate)]
         lptr, lstride = self._rows_view(lora)
         rows, R = lora.shape
         if w2.dtype != q.dtype or not w2.is_contiguous() or bias.dtype != torch.float32:
             raise KernelError("the decays read their second matrix in the path's dtype and a float32 bias")
+        chunk = self._memory_chunk(views, q.dtype, dim, vdim, False, batch)
         decays = torch.empty((rows, heads * dim), dtype=torch.float32, device=q.device)
-        self._ok(self.memory.krk_memory_decays(decays.data_ptr(), lptr, lstride, w2.data_ptr(), bias.data_ptr(), float(tau), rows,
-                                               heads * dim, R, _code(q.dtype), self._stream()), "log decays")
-        self._memory_scan(q, k, v, gate, decays, None, heads, dim, vdim, norm_w, eps, state, None, batch, out, out_col, out_scale)
+        if chunk:
+            self._ok(self.memory.krk_memory_chunk_decays(decays.data_ptr(), lptr, lstride, w2.data_ptr(), bias.data_ptr(),
+                                                         float(tau), heads * dim, R, batch.n_seqs, batch.max_q_len,
+                                                         batch.cu_q.data_ptr(), batch.seq_qlen.data_ptr(), self._stream()),
+                     "log decays summed within chunks")
+        else:
+            self._ok(self.memory.krk_memory_decays(decays.data_ptr(), lptr, lstride, w2.data_ptr(), bias.data_ptr(), float(tau),
+                                                   rows, heads * dim, R, _code(q.dtype), self._stream()), "log decays")
+        self._memory_scan(views, chunk, q.dtype, decays, None, heads, dim, vdim, norm_w, eps, state, None, batch, rows, out,
+                          out_col, out_scale)
 
     def mlstm_scan(self, q, k, v, gate, if_rows, if_bias, cap, heads, dim, vdim, norm_w, eps, state, nm, batch, out, out_col,
                    out_scale):
         """The matrix LSTM over a step's rows; ``if_rows`` [rows, 2 * heads]: input then forget gates before bias and cap;
         ``nm`` [slots, heads, dim + 1]: the vector beside the matrix and the running maximum. ``norm_w`` [heads * vdim]."""
+        views = [self._rows_view(t) for t in (q, k, v, gate)]
         zptr, zstride = self._rows_view(if_rows)
         rows = q.shape[0]
         gates = torch.empty((rows, heads, 4), dtype=torch.float32, device=q.device)
         self._ok(self.memory.krk_memory_gates(gates.data_ptr(), zptr, zstride, if_bias.data_ptr(), float(cap), nm.data_ptr(), heads,
                                               dim, batch.n_seqs, batch.max_q_len, batch.cu_q.data_ptr(), batch.seq_qlen.data_ptr(),
                                               batch.seq_slot.data_ptr(), _code(q.dtype), self._stream()), "matrix LSTM gates")
-        self._memory_scan(q, k, v, gate, None, gates, heads, dim, vdim, norm_w, eps, state, nm, batch, out, out_col, out_scale)
+        chunk = self._memory_chunk(views, q.dtype, dim, vdim, True, batch)
+        self._memory_scan(views, chunk, q.dtype, None, gates, heads, dim, vdim, norm_w, eps, state, nm, batch, rows, out, out_col,
+                          out_scale)
 
     # -- state-space mixer ------------------------------------------------------------------
     SSD_CHUNK = 128  # tokens per chunk where one sequence's step is long enough to be scanned in chunks

@@ -7,7 +7,8 @@ Kinds of library: ``core`` (kernels whose sizes are run-time arguments),
 sink or over latent rows), ``scan`` (recurrent state), ``memory`` (matrix states
 without a removal term) and ``moe`` (routed
 experts); each of the last four is compiled and loaded when a model first calls
-one of its kernels, so a model compiles what it needs. A library
+one of its kernels, so a model compiles what it needs; ``latent_k<D>_v<P>`` (prompt
+attention over keys and values made from latent rows, per pair of sizes, likewise). A library
 is rebuilt when a source or a flag changes (its name carries a hash of both) and
 is otherwise loaded as it is. Libraries live in ``csrc/_build`` inside the
 package when that is writable, else under ``$KRK_BUILD_DIR`` or a per-user
@@ -35,9 +36,10 @@ CORE_SOURCES = ["elementwise.cu", "rope_kv.cu", "gemm_simple.cu", "select.cu", "
 CORE_LIBS = ["-lcublasLt"]  # lt_gemm.cu; the process already holds the copy that torch loaded
 MIX_SOURCES = ["wide_rows.cu", "sink_attention.cu", "latent.cu", "hyper.cu", "mixed_attention.cu"]
 SCAN_SOURCES = ["recurrent.cu", "ssd.cu"]
-MEMORY_SOURCES = ["matrix_memory.cu"]
+MEMORY_SOURCES = ["matrix_memory.cu", "matrix_memory_chunks.cu"]
 MOE_SOURCES = ["routed.cu"]
 SMALL_LIBRARIES = {"mix": MIX_SOURCES, "scan": SCAN_SOURCES, "memory": MEMORY_SOURCES, "moe": MOE_SOURCES}
+LATENT_SOURCES = ["latent_prefill.cu"]
 ATTN_SOURCES = ["attention_simple.cu", "attention_mma.cu", "attention_tcgen05.cu"]
 HEADERS = ["common.cuh", "mma.cuh", "tcgen05.cuh", "attention_noalloc.h"]
 
@@ -95,7 +97,12 @@ def _key(sources, defines, libs=None) -> str:
     return h.hexdigest()[:12]
 
 
-def library_path(kind: str, head_dim: int | None = None) -> tuple[Path, list, list]:
+def library_path(kind: str, head_dim=None) -> tuple[Path, list, list]:
+    """``head_dim``: the head size of an "attn" library, the (key, value) sizes of a "latent" one."""
+    if kind == "latent":
+        sources, (key, value) = _existing(LATENT_SOURCES), (int(n) for n in head_dim)
+        defines = [f"-DKRK_KEY_DIM={key}", f"-DKRK_VALUE_DIM={value}"]
+        return build_dir() / f"libkrk_latent_k{key}_v{value}_{_key(sources, defines, [])}.so", sources, defines
     if kind == "core":
         sources, defines, stem = _existing(CORE_SOURCES), [], "libkrk_core"
     elif kind in SMALL_LIBRARIES:
@@ -113,7 +120,7 @@ def _compile_one(nvcc: str, src: Path, obj: Path, defines) -> None:
         raise BuildError(f"nvcc failed on {src.name}:\n{r.stdout}\n{r.stderr}")
 
 
-def build_library(kind: str, head_dim: int | None = None, verbose: bool = True) -> Path:
+def build_library(kind: str, head_dim=None, verbose: bool = True) -> Path:
     """Return the path of the library, compiling it first if it is not there."""
     target, sources, defines = library_path(kind, head_dim)
     if target.is_file():
@@ -166,9 +173,12 @@ def build_library(kind: str, head_dim: int | None = None, verbose: bool = True) 
                 pass
 
 
-def build_all(head_dims=(16, 32, 64, 128), verbose: bool = True) -> list[Path]:
-    """Compile the core library and the attention library of every given head size."""
+def build_all(head_dims=(16, 32, 64, 128), verbose: bool = True, latent_dims=((192, 128),)) -> list[Path]:
+    """Compile the core library, the attention library of every given head size and the latent library of every given
+    pair of sizes."""
     out = [build_library("core", verbose=verbose)] + [build_library(kind, verbose=verbose) for kind in SMALL_LIBRARIES]
     for d in head_dims:
         out.append(build_library("attn", d, verbose=verbose))
+    for pair in latent_dims:
+        out.append(build_library("latent", pair, verbose=verbose))
     return out
