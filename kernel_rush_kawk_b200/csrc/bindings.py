@@ -90,6 +90,7 @@ _MOE_SIGNATURES = {
     "krk_moe_down_pairs": [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, _P, c_int, _P, c_int, _P],
     "krk_moe_sort": [_P, _P, _P, c_int, c_int, c_int, _P],
     "krk_moe_gather": [_P, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P],
+    "krk_grouped_gemm": [_P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P, _P],
     "krk_moe_combine": [_P, _P, _P, _P, _P, _P, _P, c_int, _P, c_int, c_int, c_int, _P, c_int, _P, c_int, _P],
 }
 _MEMORY_SIGNATURES = {
@@ -97,6 +98,8 @@ _MEMORY_SIGNATURES = {
     "krk_memory_decays": [_P, _P, c_int, _P, _P, c_float, c_int, c_int, c_int, c_int, _P],
     "krk_memory_scan": [_P, _P, c_int, _P, c_int, _P, c_int, c_float, _P, _P, _P, _P, c_int, c_int, c_int, c_int, _P, _P, _P,
                         c_int, _P],
+    "krk_memory_step": [_P, c_int, c_int, c_float, _P, c_int, _P, c_int, _P, c_int, _P, c_int, c_float, _P, c_int, _P, _P, c_float,
+                        c_int, _P, _P, _P, c_float, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P],
     "krk_memory_chunk_tokens": [c_int, c_int, c_int],
     "krk_memory_chunk_decays": [_P, _P, c_int, _P, _P, c_float, c_int, c_int, c_int, c_int, _P, _P, _P],
     "krk_memory_chunks": [_P, _P, c_int, _P, c_int, _P, c_int, c_float, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int,
@@ -837,6 +840,9 @@ class Kernels:
         place = torch.empty(rows * top, dtype=torch.int32, device=x.device)
         self._ok(self.moe.krk_moe_sort(offsets.data_ptr(), place.data_ptr(), experts.data_ptr(), rows, top, E,
                                        self._stream()), "expert ordering")
+        if self._use_grouped(x, K, F, C, gated):
+            return self._grouped_experts(x, w_gate_up, w_down, experts, weights, activation, add, add_gate, gated, add_input,
+                                         offsets, place)
         bounds = offsets.tolist()
         most = max(bounds[e + 1] - bounds[e] for e in range(E))
         cap = -(-most // 16) * 16
@@ -862,6 +868,34 @@ class Kernels:
                     yg[a:b] = self.linear(h, w_down[e])
         self._ok(self.moe.krk_moe_combine(out.data_ptr(), _ptr(add), _ptr(add_gate), yg.data_ptr(), place.data_ptr(), experts.data_ptr(),
                                           offsets.data_ptr(), cap, weights.data_ptr(), rows, top, C, ptr, stride,
+                                          _ptr(add_input), _code(x.dtype), self._stream()), "experts' sum")
+        return out
+
+    @staticmethod
+    def _use_grouped(x, K, F, C, gated) -> bool:
+        """Whether the experts' products of many rows run as two grouped launches (sizes and alignment)."""
+        return (not gated and x.dtype == torch.bfloat16 and K % 8 == 0 and F % 8 == 0 and C % 8 == 0 and min(K, F) >= 64)
+
+    def _grouped_experts(self, x, w_in, w_down, experts, weights, activation, add, add_gate, gated, add_input, offsets, place):
+        """``moe_experts`` for many rows with the experts' row counts left on the device: rows ordered by expert, the first
+        product (the activation in its epilogue), the second, and the weighted sum."""
+        rows, top = experts.shape
+        E, C, F = w_down.shape
+        K = x.shape[1]
+        ptr, stride = self._rows_view(x)
+        pairs = rows * top
+        empty = lambda n: torch.empty((pairs, n), dtype=x.dtype, device=x.device)
+        xg, h, yg = empty(K), empty(F), empty(C)
+        self._ok(self.moe.krk_moe_gather(xg.data_ptr(), ptr, stride, place.data_ptr(), experts.data_ptr(), offsets.data_ptr(), 0,
+                                         rows, top, K, _code(x.dtype), self._stream()), "expert gather")
+        self._ok(self.moe.krk_grouped_gemm(h.data_ptr(), xg.data_ptr(), w_in.data_ptr(), offsets.data_ptr(), pairs, E, F, K,
+                                           _ACTIVATIONS[activation], self.error.data_ptr(), self._stream()),
+                 "experts' first product")
+        self._ok(self.moe.krk_grouped_gemm(yg.data_ptr(), h.data_ptr(), w_down.data_ptr(), offsets.data_ptr(), pairs, E, C, F, -1,
+                                           self.error.data_ptr(), self._stream()), "experts' second product")
+        out = torch.empty((rows, C), dtype=x.dtype, device=x.device)
+        self._ok(self.moe.krk_moe_combine(out.data_ptr(), _ptr(add), _ptr(add_gate), yg.data_ptr(), place.data_ptr(),
+                                          experts.data_ptr(), offsets.data_ptr(), 0, weights.data_ptr(), rows, top, C, ptr, stride,
                                           _ptr(add_input), _code(x.dtype), self._stream()), "experts' sum")
         return out
 
@@ -1151,13 +1185,36 @@ class Kernels:
             return 0
         return int(self.memory.krk_memory_chunk_tokens(dim, vdim, int(gated)))
 
-    def _memory_scan(self, views, chunk, dtype, decays, gates, heads, dim, vdim, norm_w, eps, state, nm, batch, rows, out,
-                     out_col, out_scale):
+    def _memory_step(self, views, z, w2, bias, constant, heads, dim, vdim, norm_w, eps, state, nm, batch, rows, dtype, out,
+                     out_col, out_scale) -> bool:
+        """A single-token step as one launch; False where the step or the sizes are not of that kind."""
+        if not batch.is_decode or rows != batch.n_seqs or vdim > 1024 or (vdim % 4 and vdim > 256):
+            return False
+        self._check_memory_state(state, nm, heads, dim, vdim)
         optr, ostride = self._rows_view(out)
+        # blocks per (sequence, head) by the number of such items alone, so that a captured step stays valid
+        items = batch.n_seqs * heads
+        split = 8 if items <= 18 else 4 if items <= 37 else 2 if items <= 74 else 1
+        while split > 1 and vdim < 16 * split:
+            split //= 2
+        self._ok(self.memory.krk_memory_step(optr, ostride, int(out_col), float(out_scale), *views[0], *views[1], *views[2],
+                                             *views[3], float(dim) ** -0.5, *z, _ptr(w2), bias.data_ptr(), float(constant),
+                                             0 if w2 is None else w2.shape[1], state.data_ptr(), _ptr(nm), norm_w.data_ptr(),
+                                             float(eps), heads, dim, vdim, batch.n_seqs, split, batch.seq_slot.data_ptr(),
+                                             _code(dtype), self._stream()), "single-token matrix-state step")
+        return True
+
+    @staticmethod
+    def _check_memory_state(state, nm, heads, dim, vdim) -> None:
         if state.dtype != torch.float32 or not state.is_contiguous() or state.shape[1:] != (heads, dim, vdim):
             raise KernelError("the scan keeps a contiguous float32 state [slots, heads, dim, vdim]")
         if nm is not None and (nm.dtype != torch.float32 or not nm.is_contiguous() or nm.shape[1:] != (heads, dim + 1)):
             raise KernelError("the gated scan keeps a contiguous float32 [slots, heads, dim + 1] beside its state")
+
+    def _memory_scan(self, views, chunk, dtype, decays, gates, heads, dim, vdim, norm_w, eps, state, nm, batch, rows, out,
+                     out_col, out_scale):
+        optr, ostride = self._rows_view(out)
+        self._check_memory_state(state, nm, heads, dim, vdim)
         gated = nm is not None
         y = torch.empty((rows, heads * (vdim + int(gated))), dtype=torch.float32, device=self.device)
         tables = (batch.cu_q.data_ptr(), batch.seq_qlen.data_ptr(), batch.seq_slot.data_ptr())
@@ -1187,6 +1244,9 @@ class Kernels:
         rows, R = lora.shape
         if w2.dtype != q.dtype or not w2.is_contiguous() or bias.dtype != torch.float32:
             raise KernelError("the decays read their second matrix in the path's dtype and a float32 bias")
+        if self._memory_step(views, (lptr, lstride), w2, bias, tau, heads, dim, vdim, norm_w, eps, state, None, batch, rows,
+                             q.dtype, out, out_col, out_scale):
+            return
         chunk = self._memory_chunk(views, q.dtype, dim, vdim, False, batch)
         decays = torch.empty((rows, heads * dim), dtype=torch.float32, device=q.device)
         if chunk:
@@ -1207,6 +1267,9 @@ class Kernels:
         views = [self._rows_view(t) for t in (q, k, v, gate)]
         zptr, zstride = self._rows_view(if_rows)
         rows = q.shape[0]
+        if self._memory_step(views, (zptr, zstride), None, if_bias, cap, heads, dim, vdim, norm_w, eps, state, nm, batch, rows,
+                             q.dtype, out, out_col, out_scale):
+            return
         gates = torch.empty((rows, heads, 4), dtype=torch.float32, device=q.device)
         self._ok(self.memory.krk_memory_gates(gates.data_ptr(), zptr, zstride, if_bias.data_ptr(), float(cap), nm.data_ptr(), heads,
                                               dim, batch.n_seqs, batch.max_q_len, batch.cu_q.data_ptr(), batch.seq_qlen.data_ptr(),

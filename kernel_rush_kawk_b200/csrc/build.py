@@ -36,8 +36,8 @@ CORE_SOURCES = ["elementwise.cu", "rope_kv.cu", "gemm_simple.cu", "select.cu", "
 CORE_LIBS = ["-lcublasLt"]  # lt_gemm.cu; the process already holds the copy that torch loaded
 MIX_SOURCES = ["wide_rows.cu", "sink_attention.cu", "latent.cu", "hyper.cu", "mixed_attention.cu"]
 SCAN_SOURCES = ["recurrent.cu", "ssd.cu"]
-MEMORY_SOURCES = ["matrix_memory.cu", "matrix_memory_chunks.cu"]
-MOE_SOURCES = ["routed.cu"]
+MEMORY_SOURCES = ["matrix_memory.cu", "matrix_memory_chunks.cu", "matrix_memory_step.cu"]
+MOE_SOURCES = ["routed.cu", "grouped_gemm.cu"]
 SMALL_LIBRARIES = {"mix": MIX_SOURCES, "scan": SCAN_SOURCES, "memory": MEMORY_SOURCES, "moe": MOE_SOURCES}
 LATENT_SOURCES = ["latent_prefill.cu"]
 ATTN_SOURCES = ["attention_simple.cu", "attention_mma.cu", "attention_tcgen05.cu"]
