@@ -96,15 +96,15 @@ _MOE_SIGNATURES = {
 _MEMORY_SIGNATURES = {
     "krk_memory_gates": [_P, _P, c_int, _P, c_float, _P, c_int, c_int, c_int, c_int, _P, _P, _P, c_int, _P],
     "krk_memory_decays": [_P, _P, c_int, _P, _P, c_float, c_int, c_int, c_int, c_int, _P],
-    "krk_memory_scan": [_P, _P, c_int, _P, c_int, _P, c_int, c_float, _P, _P, _P, _P, c_int, c_int, c_int, c_int, _P, _P, _P,
+    "krk_memory_scan": [_P, _P, _P, c_int, _P, c_int, _P, c_int, c_float, _P, _P, _P, _P, c_int, c_int, c_int, c_int, _P, _P, _P,
                         c_int, _P],
     "krk_memory_step": [_P, c_int, c_int, c_float, _P, c_int, _P, c_int, _P, c_int, _P, c_int, c_float, _P, c_int, _P, _P, c_float,
                         c_int, _P, _P, _P, c_float, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P],
     "krk_memory_chunk_tokens": [c_int, c_int, c_int],
     "krk_memory_chunk_decays": [_P, _P, c_int, _P, _P, c_float, c_int, c_int, c_int, c_int, _P, _P, _P],
-    "krk_memory_chunks": [_P, _P, c_int, _P, c_int, _P, c_int, c_float, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int,
+    "krk_memory_chunks": [_P, _P, _P, c_int, _P, c_int, _P, c_int, c_float, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int,
                           _P, _P, _P, _P],
-    "krk_memory_finish": [_P, c_int, c_int, c_float, _P, _P, _P, c_int, _P, c_int, c_int, c_float, c_int, c_int, _P],
+    "krk_memory_finish": [_P, c_int, c_int, c_float, _P, _P, _P, _P, c_int, _P, c_int, c_int, c_float, c_int, c_int, _P],
 }
 _LATENT_SIGNATURES = {
     "krk_latent_prefill": [_P, c_int, c_float, _P, c_int, c_int, c_int, _P, _P, c_int, c_int, _P, c_float, c_float, c_int, c_int,
@@ -1216,23 +1216,24 @@ class Kernels:
         optr, ostride = self._rows_view(out)
         self._check_memory_state(state, nm, heads, dim, vdim)
         gated = nm is not None
-        y = torch.empty((rows, heads * (vdim + int(gated))), dtype=torch.float32, device=self.device)
+        y = torch.empty((rows, heads * vdim), dtype=torch.float32, device=self.device)
+        den = torch.empty((rows, heads), dtype=torch.float32, device=self.device) if gated else None
         tables = (batch.cu_q.data_ptr(), batch.seq_qlen.data_ptr(), batch.seq_slot.data_ptr())
         if chunk:
             chunks = batch.n_seqs * -(-batch.max_q_len // chunk) * heads
             cs = torch.empty((chunks, dim * (vdim + int(gated))), dtype=torch.float32, device=self.device)
             cd = torch.empty((chunks, dim), dtype=torch.float32, device=self.device)
-            self._ok(self.memory.krk_memory_chunks(y.data_ptr(), *views[0], *views[1], *views[2], float(dim) ** -0.5, _ptr(decays),
+            self._ok(self.memory.krk_memory_chunks(y.data_ptr(), _ptr(den), *views[0], *views[1], *views[2], float(dim) ** -0.5, _ptr(decays),
                                                    _ptr(gates), state.data_ptr(), _ptr(nm), cs.data_ptr(), cd.data_ptr(), heads,
                                                    dim, vdim, batch.n_seqs, batch.max_q_len, *tables, self._stream()),
                      "matrix-state scan in chunks")
             self.launches += 2
         else:
-            self._ok(self.memory.krk_memory_scan(y.data_ptr(), *views[0], *views[1], *views[2], float(dim) ** -0.5, _ptr(decays),
+            self._ok(self.memory.krk_memory_scan(y.data_ptr(), _ptr(den), *views[0], *views[1], *views[2], float(dim) ** -0.5, _ptr(decays),
                                                  _ptr(gates), state.data_ptr(), _ptr(nm), heads, dim, vdim, batch.n_seqs, *tables,
                                                  _code(dtype), self._stream()),
                      "matrix-state scan (up to 1,024 key channels a head)")
-        self._ok(self.memory.krk_memory_finish(optr, ostride, int(out_col), float(out_scale), y.data_ptr(), _ptr(gates), *views[3],
+        self._ok(self.memory.krk_memory_finish(optr, ostride, int(out_col), float(out_scale), y.data_ptr(), _ptr(den), _ptr(gates), *views[3],
                                                norm_w.data_ptr(), heads, vdim, float(eps), rows, _code(dtype), self._stream()),
                  "matrix-state head norm and gate")
 

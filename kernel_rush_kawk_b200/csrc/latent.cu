@@ -17,7 +17,7 @@
 // multiplied by sigmoid of the gate's element of the same place (heads * N columns). One block per (tile of output elements, head, tile of 8 rows): the
 // rows' slices sit in shared memory as float32, each warp owns output elements, its lanes split K
 // (coalesced reads of W's rows), sums are float32 and their order does not depend on the other rows.
-#include "common.cuh"
+#include "mma.cuh"
 
 namespace {
 
@@ -177,6 +177,64 @@ head_linear_kernel(T* __restrict__ out, int out_stride, int out_col, int out_hea
   }
 }
 
+// The same on the tensor cores for bfloat16 and K a multiple of 8: a warp takes 8 output elements of one head for up to 16
+// rows. A lane loads 16 bytes of its output element's weight row and of its two input rows: along K a lane's eight elements
+// stand for elements 2t, 2t + 1, 2t + 8, 2t + 9 of two m16n8k16 products, the same places in both operands, so no operand
+// passes through shared memory. A row's sums depend on its own elements alone.
+__global__ void __launch_bounds__(HL_WARPS * 32)
+head_linear_mma_kernel(bf16* __restrict__ out, int out_stride, int out_col, int out_head, float out_scale,
+                       const bf16* __restrict__ x, int x_stride, int x_head, const bf16* __restrict__ w, int N, int K, int rows,
+                       int rot, const float* __restrict__ inv_freq, float factor, const int* __restrict__ row_pos,
+                       const bf16* __restrict__ gate, int gate_stride) {
+  grid_launch_dependents();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int g = lane >> 2, t4 = lane & 3;
+  const int h = blockIdx.y, r0 = blockIdx.z * 16;
+  const int n0 = (blockIdx.x * HL_WARPS + warp) * 8;
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+  const bool w_on = n0 + g < N, a_on = r0 + g < rows, b_on = r0 + g + 8 < rows;
+  const bf16* wr = w + ((size_t)h * N + (w_on ? n0 + g : 0)) * K + 8 * t4;
+  const bf16* xa = x + (size_t)(r0 + g) * x_stride + (size_t)h * x_head + 8 * t4;
+  const bf16* xb = xa + (size_t)8 * x_stride;
+  constexpr int FLY = 4;
+  uint4 wv[FLY];
+#pragma unroll
+  for (int i = 0; i < FLY; ++i) wv[i] = (w_on && 32 * i + 8 * t4 < K) ? *reinterpret_cast<const uint4*>(wr + 32 * i) : zero;
+  grid_dependency_wait();  // no kernel writes the weights
+  float acc[4] = {0.f, 0.f, 0.f, 0.f};
+  if (n0 < N) {
+    for (int k0 = 0; k0 < K; k0 += 32 * FLY) {
+      uint4 next[FLY], av[FLY], bv[FLY];
+#pragma unroll
+      for (int i = 0; i < FLY; ++i) {
+        const int k = k0 + 32 * i, kn = k + 32 * FLY;
+        next[i] = (w_on && kn + 8 * t4 < K) ? *reinterpret_cast<const uint4*>(wr + kn) : zero;
+        av[i] = (a_on && k + 8 * t4 < K) ? *reinterpret_cast<const uint4*>(xa + k) : zero;
+        bv[i] = (b_on && k + 8 * t4 < K) ? *reinterpret_cast<const uint4*>(xb + k) : zero;
+      }
+#pragma unroll
+      for (int i = 0; i < FLY; ++i) {
+        if (k0 + 32 * i >= K) break;
+        mma_bf16_16816(acc, av[i].x, bv[i].x, av[i].y, bv[i].y, wv[i].x, wv[i].y);
+        mma_bf16_16816(acc, av[i].z, bv[i].z, av[i].w, bv[i].w, wv[i].z, wv[i].w);
+        wv[i] = next[i];
+      }
+    }
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+      const int r = r0 + g + 8 * (c >> 1), n = n0 + 2 * t4 + (c & 1);
+      if (r >= rows || n >= N) continue;
+      float v = acc[c] * out_scale;
+      if (gate) v *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)r * gate_stride + (size_t)h * N + n])));
+      out[(size_t)r * out_stride + out_col + (size_t)h * out_head + n] = __float2bfloat16_rn(v);
+    }
+  }
+  if (rot > 0 && blockIdx.x == 0)
+    for (int r = r0 + warp; r < min(rows, r0 + 16); r += HL_WARPS)
+      rotate_pairs_warp<bf16>(out + (size_t)r * out_stride + out_col + (size_t)h * out_head + N,
+                              x + (size_t)r * x_stride + (size_t)h * x_head + K, rot, (float)row_pos[r], inv_freq, factor, lane);
+}
+
 }  // namespace
 
 KRK_API int krk_latent_norm_write(const void* proj, int stride, int c_col, int R, const float* gain, float eps,
@@ -232,6 +290,15 @@ KRK_API int krk_head_linear(void* out, int out_stride, int out_col, int out_head
                             cudaStream_t stream) {
   if (rows == 0 || heads == 0 || N == 0) return 0;
   if (rot < 0 || (rot & 1) || (rot > 0 && (!inv_freq || !row_pos))) return -2;
+  if (dtype == KRK_DTYPE_BF16 && K % 8 == 0 && x_stride % 8 == 0 && x_head % 8 == 0 &&
+      (((uintptr_t)x | (uintptr_t)w) & 15) == 0) {
+    const int tiles = (rows + 15) / 16;
+    if (heads > 65535 || tiles > 65535) return -3;
+    const dim3 grid((unsigned)((N + 8 * HL_WARPS - 1) / (8 * HL_WARPS)), (unsigned)heads, (unsigned)tiles);
+    return (int)launch_pdl(head_linear_mma_kernel, grid, dim3(HL_WARPS * 32), 0, stream, (bf16*)out, out_stride, out_col, out_head,
+                           out_scale, (const bf16*)x, x_stride, x_head, (const bf16*)w, N, K, rows, rot, inv_freq, factor, row_pos,
+                           (const bf16*)gate, gate_stride);
+  }
   const size_t smem = (size_t)HL_ROWS * ((K + 3) & ~3) * sizeof(float);
   if (smem > 200 * 1024) return -2;
   if (smem > 48 * 1024) {

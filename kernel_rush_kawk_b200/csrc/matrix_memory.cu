@@ -121,7 +121,8 @@ struct MemArgs {
   const float4* gates;     // [rows, H]: the gated kind; or null
   float* state;            // [slots, H, N, P]
   float* nm;               // [slots, H, N + 1] (gated kind)
-  float* y;                // [rows, H, P + (gated ? 1 : 0)]
+  float* y;                // [rows, H, P]
+  float* den;              // [rows, H]: n . q (gated kind)
   int H, N, P;
   const int *cu_q, *seq_qlen, *seq_slot;
 };
@@ -199,7 +200,11 @@ __global__ void __launch_bounds__(128) memory_scan_kernel(MemArgs a, int NS) {
       }
       float y = y0 + y1;
       for (int o = PW; o < 32; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-      if (ns == 0 && p < PT) a.y[((size_t)(row0 + t0 + t) * a.H + h) * PT + p] = y;
+      if (ns == 0 && p < PT) {
+        const size_t at = (size_t)(row0 + t0 + t) * a.H + h;
+        if (p < P) a.y[at * P + p] = y;
+        else a.den[at] = y;
+      }
     }
   }
 #pragma unroll
@@ -207,34 +212,63 @@ __global__ void __launch_bounds__(128) memory_scan_kernel(MemArgs a, int NS) {
     if (st && n0 + j < N) st[(size_t)(n0 + j) * step] = s[j];
 }
 
-// one warp per (row, head). Gated: y / den, weight [H * P], gate sigmoid; else weight [P], gate silu.
-template <typename T, bool GATED>
+// one warp per (row, head), V columns a lane. Gated: y / den, weight [H * P], gate sigmoid; else weight [P], gate silu.
+template <typename T, int V> struct alignas(V * sizeof(T)) Cols { T v[V]; };
+
+template <typename T, bool GATED, int V>
 __global__ void memory_finish_kernel(T* __restrict__ out, int out_stride, int out_col, float out_scale,
-                                     const float* __restrict__ y, const float4* __restrict__ gates, const T* __restrict__ g,
-                                     int g_stride, const float* __restrict__ weight, int H, int P, float eps, int rows) {
+                                     const float* __restrict__ y, const float* __restrict__ den,
+                                     const float4* __restrict__ gates, const T* __restrict__ g, int g_stride,
+                                     const float* __restrict__ weight, int H, int P, float eps, int rows) {
   grid_launch_dependents();
   grid_dependency_wait();
   const int lane = threadIdx.x & 31;
   const long long w = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (w >= (long long)rows * H) return;
   const size_t row = (size_t)(w / H);
-  const int h = (int)(w % H), PT = P + (GATED ? 1 : 0);
-  const float* yr = y + ((size_t)row * H + h) * PT;
+  const int h = (int)(w % H);
+  const float* yr = y + (size_t)w * P;
   float inv = 1.f;
-  if (GATED) inv = 1.0f / (fmaxf(fabsf(yr[P]), expf(-gates[row * H + h].w)) + 1e-6f);
+  if (GATED) inv = 1.0f / (fmaxf(fabsf(den[w]), expf(-gates[w].w)) + 1e-6f);
   float sq = 0.f;
-  for (int p = lane; p < P; p += 32) {
-    const float o = yr[p] * inv;
-    sq += o * o;
+  for (int p = V * lane; p < P; p += V * 32) {
+    const Cols<float, V> c = *reinterpret_cast<const Cols<float, V>*>(yr + p);
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      const float o = c.v[i] * inv;
+      sq += o * o;
+    }
   }
-  const float rstd = rsqrtf(warp_sum(sq) / (float)P + eps);
+  const float factor = rsqrtf(warp_sum(sq) / (float)P + eps) * inv;
   const T* gr = g + row * g_stride + (size_t)h * P;
+  const float* wr = weight + (GATED ? (size_t)h * P : 0);
   T* o = out + row * out_stride + out_col + (size_t)h * P;
-  for (int p = lane; p < P; p += 32) {
-    const float z = to_float<T>(gr[p]);
-    const float gate = GATED ? sigmoid_f(z) : z * sigmoid_f(z);
-    o[p] = from_float<T>(yr[p] * inv * rstd * weight[GATED ? h * P + p : p] * gate * out_scale);
+  for (int p = V * lane; p < P; p += V * 32) {
+    const Cols<float, V> c = *reinterpret_cast<const Cols<float, V>*>(yr + p), wt = *reinterpret_cast<const Cols<float, V>*>(wr + p);
+    const Cols<T, V> zz = *reinterpret_cast<const Cols<T, V>*>(gr + p);
+    Cols<T, V> res;
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      const float z = to_float<T>(zz.v[i]);
+      const float gate = GATED ? sigmoid_f(z) : z * sigmoid_f(z);
+      res.v[i] = from_float<T>(c.v[i] * factor * wt.v[i] * gate * out_scale);
+    }
+    *reinterpret_cast<Cols<T, V>*>(o + p) = res;
   }
+}
+
+template <typename T>
+int launch_memory_finish(void* out, int out_stride, int out_col, float out_scale, const float* y, const float* den,
+                         const float* gates, const void* g, int g_stride, const float* weight, int H, int P, float eps, int rows,
+                         cudaStream_t stream) {
+  const dim3 grid((unsigned)(((long long)rows * H + 3) / 4));
+  const uintptr_t mask = 4 * sizeof(T) - 1;
+  const bool vec = P % 4 == 0 && ((out_stride | out_col | g_stride) & 3) == 0 && (((uintptr_t)out | (uintptr_t)g) & mask) == 0 &&
+                   (((uintptr_t)y | (uintptr_t)weight) & 15) == 0;
+  auto kern = gates ? (vec ? memory_finish_kernel<T, true, 4> : memory_finish_kernel<T, true, 1>)
+                    : (vec ? memory_finish_kernel<T, false, 4> : memory_finish_kernel<T, false, 1>);
+  return (int)launch_pdl(kern, grid, dim3(128), 0, stream, (T*)out, out_stride, out_col, out_scale, y, den, (const float4*)gates,
+                         (const T*)g, g_stride, weight, H, P, eps, rows);
 }
 
 template <typename T, bool GATED>
@@ -284,33 +318,27 @@ KRK_API int krk_memory_decays(float* out, const void* lora, int lora_stride, con
 }
 
 // gates given: the gated kind (nm too); log_decay given: per-channel decays
-KRK_API int krk_memory_scan(float* y, const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride,
+KRK_API int krk_memory_scan(float* y, float* den, const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride,
                             float q_scale, const float* log_decay, const float* gates, float* state, float* nm, int H, int N,
                             int P, int n_seqs, const int* cu_q, const int* seq_qlen, const int* seq_slot, int dtype,
                             cudaStream_t stream) {
   if (n_seqs == 0) return 0;
-  if ((log_decay == nullptr) == (gates == nullptr) || (gates && !nm)) return -2;
+  if ((log_decay == nullptr) == (gates == nullptr) || (gates && (!nm || !den))) return -2;
   MemArgs a;
   a.q = q; a.k = k; a.v = v; a.q_stride = q_stride; a.k_stride = k_stride; a.v_stride = v_stride; a.q_scale = q_scale;
-  a.log_decay = log_decay; a.gates = (const float4*)gates; a.state = state; a.nm = nm; a.y = y; a.H = H; a.N = N; a.P = P;
+  a.log_decay = log_decay; a.gates = (const float4*)gates; a.state = state; a.nm = nm; a.y = y; a.den = den; a.H = H; a.N = N; a.P = P;
   a.cu_q = cu_q; a.seq_qlen = seq_qlen; a.seq_slot = seq_slot;
   if (dtype == KRK_DTYPE_F32)
     return gates ? launch_memory_scan<float, true>(a, n_seqs, stream) : launch_memory_scan<float, false>(a, n_seqs, stream);
   return gates ? launch_memory_scan<bf16, true>(a, n_seqs, stream) : launch_memory_scan<bf16, false>(a, n_seqs, stream);
 }
 
-KRK_API int krk_memory_finish(void* out, int out_stride, int out_col, float out_scale, const float* y, const float* gates,
-                              const void* g, int g_stride, const float* weight, int H, int P, float eps, int rows, int dtype,
-                              cudaStream_t stream) {
+KRK_API int krk_memory_finish(void* out, int out_stride, int out_col, float out_scale, const float* y, const float* den,
+                              const float* gates, const void* g, int g_stride, const float* weight, int H, int P, float eps,
+                              int rows, int dtype, cudaStream_t stream) {
   if (rows == 0) return 0;
-  const long long warps = (long long)rows * H;
-  const dim3 grid((unsigned)((warps + 3) / 4));
-  const float4* g4 = (const float4*)gates;
-  if (dtype == KRK_DTYPE_F32)
-    return (int)launch_pdl(gates ? memory_finish_kernel<float, true> : memory_finish_kernel<float, false>, grid, dim3(128), 0,
-                           stream, (float*)out, out_stride, out_col, out_scale, y, g4, (const float*)g, g_stride, weight, H, P,
-                           eps, rows);
-  return (int)launch_pdl(gates ? memory_finish_kernel<bf16, true> : memory_finish_kernel<bf16, false>, grid, dim3(128), 0,
-                         stream, (bf16*)out, out_stride, out_col, out_scale, y, g4, (const bf16*)g, g_stride, weight, H, P, eps,
-                         rows);
+  if (gates && !den) return -2;
+  return dtype == KRK_DTYPE_F32
+             ? launch_memory_finish<float>(out, out_stride, out_col, out_scale, y, den, gates, g, g_stride, weight, H, P, eps, rows, stream)
+             : launch_memory_finish<bf16>(out, out_stride, out_col, out_scale, y, den, gates, g, g_stride, weight, H, P, eps, rows, stream);
 }

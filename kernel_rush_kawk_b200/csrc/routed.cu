@@ -253,9 +253,22 @@ moe_down_pairs_kernel(T* __restrict__ out, const T* __restrict__ add, const floa
   grid_dependency_wait();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int row = blockIdx.y;
-  // an absent expert's activations were never written: zeros
-  for (int i = threadIdx.x; i < top * F; i += blockDim.x)
-    as[(i / F) * F4 + i % F] = experts[(size_t)row * top + i / F] < 0 ? 0.f : to_float<T>(act_in[(size_t)row * top * F + i]);
+  // an absent expert's activations were never written, and are not read below
+  const bool pieces = sizeof(T) == 2 && (F & 7) == 0 && (reinterpret_cast<uintptr_t>(act_in) & 15) == 0;
+  for (int j = 0; j < top; ++j) {
+    if (experts[(size_t)row * top + j] < 0) continue;
+    const T* src = act_in + ((size_t)row * top + j) * F;
+    if (pieces) {
+      for (int i = 8 * threadIdx.x; i < F; i += 8 * blockDim.x) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(src + i);
+        const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
+        *reinterpret_cast<float4*>(as + j * F4 + i) = make_float4(__low2float(p[0]), __high2float(p[0]), __low2float(p[1]), __high2float(p[1]));
+        *reinterpret_cast<float4*>(as + j * F4 + i + 4) = make_float4(__low2float(p[2]), __high2float(p[2]), __low2float(p[3]), __high2float(p[3]));
+      }
+    } else {
+      for (int i = threadIdx.x; i < F; i += blockDim.x) as[j * F4 + i] = to_float<T>(src[i]);
+    }
+  }
   __syncthreads();
   for (int c = blockIdx.x * PAIR_WARPS + warp; c < C; c += gridDim.x * PAIR_WARPS) {
     float total = add ? to_float<T>(add[(size_t)row * C + c]) * (add_gate ? add_gate[row] : 1.f) : 0.f;
@@ -281,6 +294,7 @@ moe_down_pairs_kernel(T* __restrict__ out, const T* __restrict__ add, const floa
             raw[jj] = on[jj] ? *reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(wr[jj]) + k) : make_uint4(0u, 0u, 0u, 0u);
 #pragma unroll
           for (int jj = 0; jj < 4; ++jj) {
+            if (!on[jj]) continue;
             const float* xs = as + min(j0 + jj, top - 1) * F4 + k;
             const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw[jj]);
             const float4 a = *reinterpret_cast<const float4*>(xs), b = *reinterpret_cast<const float4*>(xs + 4);
@@ -303,33 +317,62 @@ moe_down_pairs_kernel(T* __restrict__ out, const T* __restrict__ add, const floa
   }
 }
 
-// One block: counts per expert, offsets, each pair's place in the expert order (stable: pairs of one expert
-// keep their order), and the rows of x gathered in that order.
+// One block: counts per expert, offsets, each pair's place in the expert order (stable: pairs of one expert keep their
+// order). Every warp owns a run of the pairs and a row of counters; 32 pairs at a time, lanes with one expert find one
+// another and their rank (match), so a warp walks its run twice, once to count and once to place.
 __global__ void moe_sort_kernel(int* __restrict__ offsets, int* __restrict__ place, const int* __restrict__ experts,
                                 int pairs, int E) {
-  extern __shared__ int cnt[];  // [E + 1]
+  extern __shared__ int cnt[];  // [warps][E], then [E + 1]
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+  int* mine = cnt + (size_t)warp * E;
+  int* base = cnt + (size_t)n_warps * E;
+  for (int i = threadIdx.x; i < n_warps * E; i += blockDim.x) cnt[i] = 0;
   grid_dependency_wait();
-  for (int e = threadIdx.x; e <= E; e += blockDim.x) cnt[e] = 0;
   __syncthreads();
-  for (int i = threadIdx.x; i < pairs; i += blockDim.x)
-    if (experts[i] >= 0) atomicAdd(&cnt[experts[i] + 1], 1);
-  __syncthreads();
-  if (threadIdx.x == 0) {
-    for (int e = 0; e < E; ++e) cnt[e + 1] += cnt[e];
-    for (int e = 0; e <= E; ++e) offsets[e] = cnt[e];
+  const int run = ((pairs + n_warps - 1) / n_warps + 31) / 32 * 32;
+  const int lo = warp * run, hi = min(pairs, lo + run);
+  for (int i0 = lo; i0 < hi; i0 += 32) {
+    const int e = i0 + lane < hi ? experts[i0 + lane] : -1;
+    const unsigned same = __match_any_sync(0xffffffffu, e);
+    if (e >= 0 && lane == __ffs(same) - 1) mine[e] += __popc(same);
+    __syncwarp();
   }
   __syncthreads();
-  // a warp per expert walks the pairs in order, 32 at a time (a ballot gives each hit its rank): stable
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
-  for (int e = warp; e < E; e += n_warps) {
-    int at = cnt[e];
-    for (int i0 = 0; i0 < pairs; i0 += 32) {
-      const int i = i0 + lane;
-      const bool hit = i < pairs && experts[i] == e;
-      const unsigned mask = __ballot_sync(0xffffffffu, hit);
-      if (hit) place[i] = at + __popc(mask & ((1u << lane) - 1u));
-      at += __popc(mask);
+  // per expert: what the warps before counted; the total goes to base
+  for (int e = threadIdx.x; e < E; e += blockDim.x) {
+    int before = 0;
+    for (int w = 0; w < n_warps; ++w) {
+      const int c = cnt[(size_t)w * E + e];
+      cnt[(size_t)w * E + e] = before;
+      before += c;
     }
+    base[e] = before;
+  }
+  __syncthreads();
+  if (warp == 0) {  // totals to offsets
+    int carry = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      const int c = e0 + lane < E ? base[e0 + lane] : 0;
+      int incl = c;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int p = __shfl_up_sync(0xffffffffu, incl, o);
+        if (lane >= o) incl += p;
+      }
+      if (e0 + lane < E) base[e0 + lane] = offsets[e0 + lane] = carry + incl - c;
+      carry += __shfl_sync(0xffffffffu, incl, 31);
+    }
+    if (lane == 0) offsets[E] = carry;
+  }
+  __syncthreads();
+  for (int i0 = lo; i0 < hi; i0 += 32) {
+    const int i = i0 + lane;
+    const int e = i < hi ? experts[i] : -1;
+    const unsigned same = __match_any_sync(0xffffffffu, e);
+    if (e >= 0) place[i] = base[e] + mine[e] + __popc(same & ((1u << lane) - 1u));
+    __syncwarp();
+    if (e >= 0 && lane == __ffs(same) - 1) mine[e] += __popc(same);
+    __syncwarp();
   }
 }
 
@@ -372,6 +415,37 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const T* __restrict__ ad
     src_w[threadIdx.x] = weights[(size_t)row * top + threadIdx.x];
   }
   __syncthreads();
+  if (sizeof(T) == 2 && (C & 7) == 0 && (x_stride & 7) == 0 &&
+      ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(add) | reinterpret_cast<uintptr_t>(yg) |
+        reinterpret_cast<uintptr_t>(x)) & 15) == 0) {
+    // eight columns a thread, four chosen experts' pieces in flight; the sum in the order of the choice
+    const float ag = add ? (add_gate ? add_gate[row] : 1.f) : 0.f, px = passed ? passed[row] : 0.f;
+    auto fma8 = [](float (&t)[8], float w, const uint4& raw) {
+      const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+      for (int q = 0; q < 4; ++q) { t[2 * q] += w * __low2float(p[q]); t[2 * q + 1] += w * __high2float(p[q]); }
+    };
+    for (int c = 8 * threadIdx.x; c < C; c += 8 * blockDim.x) {
+      float t[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      if (add) fma8(t, ag, *reinterpret_cast<const uint4*>(add + (size_t)row * C + c));
+      if (passed) fma8(t, px, *reinterpret_cast<const uint4*>(x + (size_t)row * x_stride + c));
+      for (int j0 = 0; j0 < top; j0 += 4) {
+        uint4 raw[4];
+#pragma unroll
+        for (int q = 0; q < 4; ++q)
+          if (j0 + q < top && src_row[j0 + q] >= 0) raw[q] = *reinterpret_cast<const uint4*>(yg + (size_t)src_row[j0 + q] * C + c);
+#pragma unroll
+        for (int q = 0; q < 4; ++q)
+          if (j0 + q < top && src_row[j0 + q] >= 0) fma8(t, src_w[j0 + q], raw[q]);
+      }
+      uint4 o;
+      __nv_bfloat162* po = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+      for (int q = 0; q < 4; ++q) po[q] = __floats2bfloat162_rn(t[2 * q], t[2 * q + 1]);
+      *reinterpret_cast<uint4*>(out + (size_t)row * C + c) = o;
+    }
+    return;
+  }
   for (int c = threadIdx.x; c < C; c += blockDim.x) {
     float total = add ? to_float<T>(add[(size_t)row * C + c]) * (add_gate ? add_gate[row] : 1.f) : 0.f;
     if (passed) total += passed[row] * to_float<T>(x[(size_t)row * x_stride + c]);
@@ -459,8 +533,12 @@ KRK_API int krk_moe_down_pairs(void* out, const void* add, const float* add_gate
 
 KRK_API int krk_moe_sort(int* offsets, int* place, const int* experts, int rows, int top, int E, cudaStream_t stream) {
   if (rows == 0) return 0;
-  return (int)launch_pdl(moe_sort_kernel, dim3(1), dim3(1024), (size_t)(E + 1) * sizeof(int), stream, offsets, place,
-                         experts, rows * top, E);
+  int warps = 32;
+  while (warps > 1 && (size_t)(warps + 1) * E * sizeof(int) > 200 * 1024) warps >>= 1;
+  const size_t smem = (size_t)(warps + 1) * E * sizeof(int);
+  if (smem > 200 * 1024) return -2;
+  if (smem > 48 * 1024) cudaFuncSetAttribute(moe_sort_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  return (int)launch_pdl(moe_sort_kernel, dim3(1), dim3(warps * 32), smem, stream, offsets, place, experts, rows * top, E);
 }
 
 KRK_API int krk_moe_gather(void* xg, const void* x, int x_stride, const int* place, const int* experts, const int* offsets,

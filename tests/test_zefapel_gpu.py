@@ -385,12 +385,14 @@ def test_latent_attention_finds_one_loud_key_wherever_it_sits(dtype, scaled):
 MOE_SHAPES = [  # hidden, experts, identity, top, ff, (groups, keep), shared ff
     (64, 5, 3, 3, 40, (4, 2), 24), (96, 7, 1, 8, 32, (1, 1), 40), (50, 3, 3, 1, 9, (1, 1), None), (50, 5, 0, 5, 11, (1, 1), 11),
     (64, 12, 4, 2, 48, (2, 1), 64), (32, 4, 2, 2, 24, (3, 2), None), (32, 9, 0, 8, 1800, (3, 3), 8), (64, 2, 30, 4, 16, (8, 3), 16),
+    # rows ordered by expert and multiplied in one launch: experts with more than a tile of rows and with none
+    (96, 7, 1, 3, 72, (2, 1), 40), (256, 12, 4, 2, 64, (2, 1), 96), (136, 40, 8, 4, 264, (4, 2), None), (64, 70, 2, 2, 64, (6, 2), 8),
 ]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("shape", MOE_SHAPES)
-@pytest.mark.parametrize("rows", [1, 5, 200])
+@pytest.mark.parametrize("rows", [1, 5, 200, 777])
 def test_routed_experts_with_identity_experts_alone(dtype, shape, rows):
     from kernel_rush_kawk_b200.parts import RoutedExperts
 
@@ -413,6 +415,44 @@ def test_routed_experts_with_identity_experts_alone(dtype, shape, rows):
     for decode in (False, True):
         ctx = SimpleNamespace(ops=rt.ops, batch=SimpleNamespace(is_decode=decode))
         close(part.forward(ctx, h.cuda()), want, dtype, f"experts {shape}, {rows} rows, single-token step {decode}")
+
+
+def test_grouped_products_where_experts_have_few_rows_many_or_none():
+    rt = runtime(torch.bfloat16)
+    for E, N, K, counts in ((5, 200, 72, [0, 300, 1, 0, 128]), (3, 64, 128, [129, 0, 0]), (40, 320, 96, [7 * (e % 3) for e in range(40)])):
+        offsets = torch.tensor([0] + counts).cumsum(0).to(torch.int32)
+        rows = int(offsets[-1])
+        a, w = rand((rows + 5, K), 1).to(torch.bfloat16), rand((E, N, K), 2, K ** -0.5).to(torch.bfloat16)
+        for act in (-1, 5):
+            out = torch.full((rows + 5, N), 7.0, dtype=torch.bfloat16, device="cuda")
+            a_d, w_d, o_d = a.cuda(), w.cuda(), offsets.cuda()
+            rt.ops._ok(rt.ops.moe.krk_grouped_gemm(out.data_ptr(), a_d.data_ptr(), w_d.data_ptr(), o_d.data_ptr(), rows + 5, E, N, K,
+                                                   act, rt.ops.error.data_ptr(), rt.ops._stream()), "grouped product")
+            want = torch.full((rows + 5, N), 7.0, dtype=torch.float64)
+            for e in range(E):
+                lo, hi = int(offsets[e]), int(offsets[e + 1])
+                y = a[lo:hi].double() @ w[e].double().t()
+                want[lo:hi] = torch.clamp(y, min=0.0) ** 2 if act == 5 else y
+            close(out, want, torch.bfloat16, f"{E} experts, act {act}")  # rows beyond the last expert's stay as they were
+    rt.ops.check()
+
+
+def test_experts_are_ordered_stably():
+    rt = runtime(torch.float32)
+    g = torch.Generator().manual_seed(3)
+    for rows, top, E in ((1, 2, 3), (700, 3, 11), (2048, 6, 64), (33, 1, 300)):
+        experts = torch.randint(-1, E, (rows, top), generator=g, dtype=torch.int32)
+        offsets = torch.empty(E + 1, dtype=torch.int32, device="cuda")
+        place = torch.full((rows * top,), -5, dtype=torch.int32, device="cuda")
+        d = experts.cuda()
+        rt.ops._ok(rt.ops.moe.krk_moe_sort(offsets.data_ptr(), place.data_ptr(), d.data_ptr(), rows, top, E, rt.ops._stream()), "ordering")
+        flat = experts.flatten()
+        counts = torch.bincount(flat[flat >= 0].long(), minlength=E)
+        assert offsets.tolist() == [0] + counts.cumsum(0).tolist()
+        order = sorted((i for i in range(flat.numel()) if flat[i] >= 0), key=lambda i: (int(flat[i]), i))
+        want = torch.full((flat.numel(),), -5, dtype=torch.int32)
+        want[torch.tensor(order, dtype=torch.long)] = torch.arange(len(order), dtype=torch.int32)
+        assert torch.equal(place.cpu(), want)
 
 
 def test_routing_within_groups_by_hand():
