@@ -70,6 +70,7 @@ _MIX_SIGNATURES = {
                         _P, _P, c_int, c_int, _P],
     "krk_latent_rows": [_P, _P, c_int, c_int, c_int, _P, c_int, c_int, _P, c_int, _P, c_float, c_float, _P, _P, _P, _P, c_int,
                         _P, c_int, c_int, _P],
+    "krk_latent_decode": [_P, _P, _P, c_int, c_int, c_int, c_int, _P, _P, _P, c_int, _P, c_float, c_int, c_int, _P],
     "krk_latent_gather": [_P, _P, c_int, c_int, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P],
     "krk_embed_bigram": [_P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_longlong, c_longlong, _P, _P, _P, _P, _P, c_int, _P],
     "krk_bias_norm_rotate_write": [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_float, _P, c_int,
@@ -334,7 +335,7 @@ class Kernels:
         self._ok(self.core.krk_skinny_linear(
             out.data_ptr(), src.data_ptr(), w.data_ptr(), _ptr(branch), _ptr(gain), _ptr(x_new),
             int(gain is not None and gain.dtype == torch.float32), None, M, N, K, float(x.eps) if lazy else float(act_limit),
-            int(gate_act if swiglu_rows > 0 else 0), _code(out_dtype), self._stream()), "skinny product")
+            int(gate_act if swiglu_rows > 0 or gate_act == 4 else 0), _code(out_dtype), self._stream()), "skinny product")
         if lazy:
             x.mark_fused()
         return out
@@ -716,10 +717,30 @@ class Kernels:
                                           R, D, rows, E, m.inv_freq.data_ptr(), float(m.rot_factor), batch.row_pos.data_ptr(),
                                           None, 0, _code(q.dtype), self._stream()), "queries into the latent space")
         mixed = torch.empty((rows, H * R), dtype=q.dtype, device=q.device)
-        self.sink_attention(qx, 0, H, W, R, None, m.scale, None, batch, cache, mixed, 0, 1.0)
+        if not self._latent_decode(qx, H, R, W, m.scale, batch, cache, mixed):
+            self.sink_attention(qx, 0, H, W, R, None, m.scale, None, batch, cache, mixed, 0, 1.0)
         self._ok(self.mix.krk_head_linear(optr, ostride, int(out_col), P, float(out_scale), mixed.data_ptr(), H * R, R,
                                           m.uv.data_ptr(), H, P, R, rows, 0, None, 1.0, None, g_ptr, g_stride, _code(q.dtype),
                                           self._stream()), "values out of the latent space")
+
+    def _latent_decode(self, qx, H, R, W, scale, batch, cache, mixed) -> bool:
+        """A single-token step in bfloat16 on the tensor cores; False where the step or the sizes are not of that kind."""
+        if not batch.is_decode or qx.dtype != torch.bfloat16 or R % 16 or W % 16 or R > 512:
+            return False
+        # blocks that share a sequence's pages by the step's shape alone, so that a captured step stays valid
+        splits = max(1, min(32, 148 // (batch.n_seqs * -(-H // 16))))
+        key = ("latent", batch.n_seqs, H, R, splits)
+        scratch = self._partials.get(key)
+        if scratch is None:
+            scratch = self._partials[key] = torch.empty(batch.n_seqs * H * splits * (R + 2), dtype=torch.float32, device=self.device)
+        rc = self.mix.krk_latent_decode(mixed.data_ptr(), scratch.data_ptr(), qx.data_ptr(), qx.stride(0), H, R, W,
+                                        batch.seq_slot.data_ptr(), batch.seq_start.data_ptr(), cache.table.data_ptr(), cache.width,
+                                        cache.k.data_ptr(), float(scale), splits, batch.n_seqs, self._stream())
+        if rc == -2:
+            return False
+        self._ok(rc, "single-token attention over latent rows")
+        self.launches += 1
+        return True
 
     LATENT_DENSE_BYTES = 4 << 30  # keys and values of a step's whole context beyond this size are not written out
 
@@ -810,7 +831,9 @@ class Kernels:
         return experts, weights, row_gate, passed
 
     def up_act(self, h, w_up, activation):
-        """act(up h), without a gate."""
+        """act(up h), without a gate; the squared relu of few bfloat16 rows runs in the product's epilogue."""
+        if activation == "relu2" and self._use_skinny(h, w_up):
+            return self._skinny(self._resolve(h), w_up, w_up.dtype, gate_act=4)
         return self.act_rows(self.linear(h, w_up), activation)
 
     def moe_experts(self, x, w_gate_up, w_down, experts, weights, intermediate, activation, add=None, add_gate=None,

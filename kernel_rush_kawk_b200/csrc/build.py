@@ -34,7 +34,7 @@ SRC_DIR = Path(__file__).parent
 
 CORE_SOURCES = ["elementwise.cu", "rope_kv.cu", "gemm_simple.cu", "select.cu", "skinny_bf16.cu", "gemm_tcgen05.cu", "lt_gemm.cu"]
 CORE_LIBS = ["-lcublasLt"]  # lt_gemm.cu; the process already holds the copy that torch loaded
-MIX_SOURCES = ["wide_rows.cu", "sink_attention.cu", "latent.cu", "hyper.cu", "mixed_attention.cu"]
+MIX_SOURCES = ["wide_rows.cu", "sink_attention.cu", "latent.cu", "hyper.cu", "mixed_attention.cu", "latent_decode.cu"]
 SCAN_SOURCES = ["recurrent.cu", "ssd.cu"]
 MEMORY_SOURCES = ["matrix_memory.cu", "matrix_memory_chunks.cu", "matrix_memory_step.cu"]
 MOE_SOURCES = ["routed.cu", "grouped_gemm.cu"]

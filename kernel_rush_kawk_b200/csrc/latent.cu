@@ -80,6 +80,47 @@ template <typename T>
 __device__ __forceinline__ void rms_row_warp(T* dst, const T* __restrict__ src, int n, const float* __restrict__ gain, float eps,
                                              int lane) {
   float sq = 0.f;
+  if (sizeof(T) == 2 && (n & 7) == 0 &&
+      ((reinterpret_cast<uintptr_t>(src) | reinterpret_cast<uintptr_t>(dst) | reinterpret_cast<uintptr_t>(gain)) & 15) == 0) {
+    // 16-byte pieces, the first eight a lane kept in registers between the sum and the result (rows of up to 2,048)
+    constexpr int KEEP = 8;
+    uint4 raw[KEEP];
+    auto squares = [](const uint4& r) {
+      const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&r);
+      float t = 0.f;
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const float a = __low2float(p[q]), b = __high2float(p[q]);
+        t += a * a + b * b;
+      }
+      return t;
+    };
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+      const int i = 8 * (lane + 32 * j);
+      raw[j] = i < n ? *reinterpret_cast<const uint4*>(src + i) : make_uint4(0u, 0u, 0u, 0u);
+    }
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) sq += squares(raw[j]);
+    for (int i = 8 * (lane + 32 * KEEP); i < n; i += 256) sq += squares(*reinterpret_cast<const uint4*>(src + i));
+    const float rstd = rsqrtf(warp_sum(sq) / (float)n + eps);
+    auto store = [&](int i, const uint4& r) {
+      const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&r);
+      uint4 o;
+      __nv_bfloat162* po = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+      for (int q = 0; q < 4; ++q)
+        po[q] = __floats2bfloat162_rn(__low2float(p[q]) * rstd * gain[i + 2 * q], __high2float(p[q]) * rstd * gain[i + 2 * q + 1]);
+      *reinterpret_cast<uint4*>(dst + i) = o;
+    };
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+      const int i = 8 * (lane + 32 * j);
+      if (i < n) store(i, raw[j]);
+    }
+    for (int i = 8 * (lane + 32 * KEEP); i < n; i += 256) store(i, *reinterpret_cast<const uint4*>(src + i));
+    return;
+  }
   for (int i = lane; i < n; i += 32) {
     const float f = to_float<T>(src[i]);
     sq += f * f;

@@ -311,6 +311,9 @@ skinny_kernel(TOut* __restrict__ out, const bf16* __restrict__ x, const bf16* __
       } else if (SWIGLU) {
         const float gate = round_to<bf16>(v), up = round_to<bf16>(v2);
         v = round_to<bf16>(gate / (1.0f + expf(-gate))) * up;
+      } else if (!NORM && eps < 0.f) {  // squared relu of the product as it would have been stored; no norm: eps is free
+        v = round_to<bf16>(v);
+        v = v > 0.f ? v * v : 0.f;
       }
       out[(size_t)m * N + n] = from_float<TOut>(v);
     }
@@ -437,6 +440,11 @@ KRK_API int krk_skinny_linear(void* out, const void* x, const void* W, const voi
   if (M > 16 || K % CHUNK || K <= 0) return -2;
   if (branch && !gain) return -2;
   const bool norm = gain != nullptr;
+  if (swiglu == 4) {  // no gate: the squared relu of the plain product; no norm prologue
+    if (out_dtype != KRK_DTYPE_BF16 || norm) return -4;
+    return pick_nt<0, false, bf16>(out, x, W, branch, gain, gain_f32, x_new, M, N, K, -1.f, stream);
+  }
+  if (!norm && !swiglu) eps = 0.f;
   if (swiglu == 2) {  // gate and up with the tanh form of GELU; no norm prologue with it
     if (out_dtype != KRK_DTYPE_BF16 || norm) return -4;
     return pick_nt<2, false, bf16>(out, x, W, branch, gain, gain_f32, x_new, M, N, K, eps, stream);

@@ -178,3 +178,13 @@ def test_presets_build_their_plans_and_are_served_by_name():
         cfg = preset_config(name)
         assert PartTree(get_architecture("Zefapel").plan(cfg), 64).expected_tensors()
     assert "zefapel_tiny" in ZefapelConfig.preset_names()
+
+
+def test_command_line_writes_a_preset_as_a_model_folder(tmp_path):
+    from kernel_rush_kawk_b200 import cli, read_config
+
+    assert cli.main(["write-random", "--preset", "zefapel_tiny", "--seed", "1", "--out", str(tmp_path / "m")]) == 0
+    arch, cfg = read_config(tmp_path / "m")
+    assert arch.name == "Zefapel" and len(cfg.layers) == 4
+    steps = list(cpu_engine(tmp_path / "m", max_tokens=256, max_context=256).generate([[5, 6, 7], [9]], 3))
+    assert len(steps) == 3 and all(len(s) == 2 for s in steps)

@@ -348,6 +348,32 @@ def test_latent_attention_alone(dtype, shape):
         close(run_part(part, rt, h, pieces, dtype, prior=[(rand((200, shape[0]), 2), [200])]), want, dtype, f"latent {shape}, pieces {pieces[:4]}")
 
 
+@pytest.mark.parametrize("heads, rank, rot", [(16, 512, 64), (5, 64, 16), (33, 128, 32), (20, 272, 16), (3, 96, 32)])
+@pytest.mark.parametrize("lengths", [[1, 64, 65, 500], [129], [2000] + [3] * 11])
+def test_single_tokens_over_latent_rows_on_the_tensor_cores(heads, rank, rot, lengths):
+    """The kernel against the general one (bfloat16, same rows): pages shared by more blocks than there are pages, sequences of
+    very different length side by side, heads that do not fill a tile."""
+    from kernel_rush_kawk_b200.cache import SequenceCache
+    from kernel_rush_kawk_b200.parts import KVNeed
+
+    rt = runtime(torch.bfloat16)
+    W = rank + rot
+    cache = SequenceCache([KVNeed(1, W, None, values=False)], 64 * 80, len(lengths), 4096, rt.device, torch.bfloat16)
+    slots = [cache.alloc() for _ in lengths]
+    for s, n in zip(slots, lengths):
+        cache.reserve(s, n)
+        cache.advance(s, n - 1)
+    cache.sync()
+    view = cache.view(0)
+    view.k.copy_(rand(tuple(view.k.shape), 1).to(torch.bfloat16))
+    batch = context(rt, slots, [n - 1 for n in lengths], [1] * len(lengths), cache).batch
+    q = rand((len(lengths), heads * W), 2, 3.0 * W ** -0.5).to(torch.bfloat16).cuda()
+    got, want = (torch.zeros((len(lengths), heads * rank), dtype=torch.bfloat16, device="cuda") for _ in range(2))
+    assert rt.ops._latent_decode(q, heads, rank, W, 0.7, batch, view, got)
+    rt.ops.sink_attention(q, 0, heads, W, rank, None, 0.7, None, batch, view, want, 0, 1.0)
+    close(got, want, torch.bfloat16, f"{heads} heads, rank {rank}, lengths {lengths[:4]}", loosen=0.3)
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_latent_attention_over_another_layers_rows(dtype):
     """The reader has head counts, sizes and weights of its own; the rows are the other part's."""
@@ -476,6 +502,10 @@ def test_squared_relu_without_a_gate(dtype):
     rt = runtime(dtype)
     z = rand((9, 200), 2, 1.5).to(dtype)
     close(rt.ops.act_rows(z.cuda(), "relu2"), torch.clamp(z.double(), min=0.0) ** 2, dtype, "squared relu")
+    for rows, K, N in ((1, 64, 40), (8, 96, 4000), (13, 256, 24), (40, 64, 48), (3, 50, 21)):  # few rows: in the product's epilogue
+        h, w = rand((rows, K), 3).to(dtype), rand((N, K), 4, K ** -0.5).to(dtype)
+        want = torch.clamp(h.double() @ w.double().t(), min=0.0) ** 2
+        close(rt.ops.up_act(h.cuda(), w.cuda(), "relu2"), want, dtype, f"squared relu of a product of {rows} rows")
 
 
 # ----------------------------------------------------------------------------------------------
@@ -585,3 +615,18 @@ def test_trace_replay_serves_the_design(folders, tmp_path):
     for t in range(10):
         row = torch.from_numpy(np.fromfile(tmp_path / "o" / f"{1 + t}.f32", dtype="<f4").reshape(1, -1))
         assert_logits(row, ref_a[60 + t:61 + t], "float32", f"replayed token {t}")
+
+
+def test_command_line_writes_a_random_model_and_generates_from_it(tmp_path, capsys):
+    """`write-random`, then `generate` from that folder and straight from the preset's name: the same weights, so the same
+    greedy tokens."""
+    from kernel_rush_kawk_b200 import cli
+
+    assert cli.main(["write-random", "--preset", "zefapel_tiny", "--seed", "3", "--out", str(tmp_path / "m")]) == 0
+    capsys.readouterr()
+    common = ["--prompt-ids", "5,6,7,8,9", "--prompt-ids", "11", "--max-new-tokens", "6", "--max-context", "256"]
+    assert cli.main(["generate", "--model", str(tmp_path / "m")] + common) == 0
+    from_folder = [json.loads(line) for line in capsys.readouterr().out.strip().splitlines()]
+    assert cli.main(["generate", "--random", "zefapel_tiny", "--weights-seed", "3"] + common) == 0
+    from_preset = [json.loads(line) for line in capsys.readouterr().out.strip().splitlines()]
+    assert from_folder == from_preset and [len(r["tokens"]) for r in from_folder] == [6, 6]
