@@ -1271,7 +1271,7 @@ class Kernels:
         if self._memory_step(views, (lptr, lstride), w2, bias, tau, heads, dim, vdim, norm_w, eps, state, None, batch, rows,
                              q.dtype, out, out_col, out_scale):
             return
-        chunk = self._memory_chunk(views, q.dtype, dim, vdim, False, batch)
+        chunk = self._memory_chunk(views, q.dtype, dim, vdim, False, batch) if R <= 192 else 0  # a chunk's rows in shared memory
         decays = torch.empty((rows, heads * dim), dtype=torch.float32, device=q.device)
         if chunk:
             self._ok(self.memory.krk_memory_chunk_decays(decays.data_ptr(), lptr, lstride, w2.data_ptr(), bias.data_ptr(),

@@ -35,6 +35,7 @@ namespace {
 
 constexpr int MAX_V_PER_LANE = 8;    // value heads up to 256
 constexpr int WIDE_V_PER_LANE = 16;  // the general kernel's second form: value rows up to 512 (latent rows)
+constexpr int WIDEST_V_PER_LANE = 32;  // its third form: up to 1,024
 
 __device__ __forceinline__ float sigmoidf_(float z) { return 1.0f / (1.0f + expf(-z)); }  // value heads up to 256
 
@@ -568,19 +569,19 @@ KRK_API int krk_sink_attention(void* out, int out_stride, int out_col, float out
                                const void* gate, int gate_stride, int gate_col, int gate_mode, int dtype,
                                cudaStream_t stream) {
   if (rows == 0) return 0;
-  if (DV > 32 * WIDE_V_PER_LANE || D > 2048) return -2;
+  if (DV > 32 * WIDEST_V_PER_LANE || D > 2048) return -2;
   const long long items = (long long)rows * HQ;
   const int warps = 4;
   const long long blocks = (items + warps - 1) / warps;
   if (blocks > 0x7fffffffLL) return -3;
   const size_t smem = (size_t)warps * D * sizeof(float);
-  const bool wide = DV > 32 * MAX_V_PER_LANE;
+  const bool wide = DV > 32 * MAX_V_PER_LANE, widest = DV > 32 * WIDE_V_PER_LANE;
   if (dtype == KRK_DTYPE_F32)
-    return (int)launch_pdl(wide ? sink_attention_kernel<float, WIDE_V_PER_LANE> : sink_attention_kernel<float, MAX_V_PER_LANE>, dim3((unsigned)blocks), dim3(warps * 32), smem, stream,
+    return (int)launch_pdl(widest ? sink_attention_kernel<float, WIDEST_V_PER_LANE> : wide ? sink_attention_kernel<float, WIDE_V_PER_LANE> : sink_attention_kernel<float, MAX_V_PER_LANE>, dim3((unsigned)blocks), dim3(warps * 32), smem, stream,
                            (float*)out, out_stride, out_col, out_scale, (const float*)proj, stride, q_col, HQ, HKV, D, DV,
                            sink, row_seq, row_pos, seq_slot, table, width, (const float*)k_cache, (const float*)v_cache,
                            v_pitch, rows, scale, window, keep_first, keep_pages, (const float*)gate, gate_stride, gate_col, gate_mode);
-  return (int)launch_pdl(wide ? sink_attention_kernel<bf16, WIDE_V_PER_LANE> : sink_attention_kernel<bf16, MAX_V_PER_LANE>,
+  return (int)launch_pdl(widest ? sink_attention_kernel<bf16, WIDEST_V_PER_LANE> : wide ? sink_attention_kernel<bf16, WIDE_V_PER_LANE> : sink_attention_kernel<bf16, MAX_V_PER_LANE>,
                          dim3((unsigned)blocks), dim3(warps * 32), smem, stream, (bf16*)out,
                          out_stride, out_col, out_scale, (const bf16*)proj, stride, q_col, HQ, HKV, D, DV, sink, row_seq,
                          row_pos, seq_slot, table, width, (const bf16*)k_cache, (const bf16*)v_cache, v_pitch, rows, scale, window,

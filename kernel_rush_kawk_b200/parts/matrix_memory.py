@@ -3,14 +3,14 @@
 Per head S is N x P (``dim`` x ``vdim``), 32-bit, zero at the start of a sequence and carried from token to token;
 q = Wq h / sqrt(N), k = Wk h, v = Wv h.
 
-* ``GatedLinearAttention`` (kind "gla"): a decay per key channel, alpha = sigmoid(z)^(1/tau) with
-  z = Wa2 (Wa1 h) + b; S <- diag(alpha) S + k v^T, o = S^T q. Each head's o goes through an RMS norm with one weight of
-  size P that the heads share; the heads side by side are multiplied by silu(Wg h) and projected.
-* ``MatrixLSTM`` (kind "mlstm"): per head a log input gate i = cap tanh((Wi h + bi) / cap) and a log forget gate
-  f = logsigmoid(cap tanh((Wf h + bf) / cap)). With a running maximum m (zero at the start), m' = max(f + m, i):
+* ``GatedLinearAttention`` (kind "gla"): row n of S decays by alpha_n = exp(logsigmoid(z_n) / tau), z = Wa2 (Wa1 h) + b;
+  S <- diag(alpha) S + k v^T, o = S^T q. The readout of every head passes an RMS norm whose weight (P numbers) is one for
+  all heads; then silu(Wg h) times that, side by side, is projected.
+* ``MatrixLSTM`` (kind "mlstm"): with c(x) = cap tanh(x / cap), a head's log gates are i = c(Wi h + bi) for the input and
+  f = logsigmoid(c(Wf h + bf)) for what is kept. With a running maximum m (zero at the start), m' = max(f + m, i):
   S <- exp(f + m - m') S + exp(i - m') k v^T, n <- exp(f + m - m') n + exp(i - m') k,
-  o = S^T q / (max(|n . q|, exp(-m')) + 1e-6). Each head's o is divided by its root mean square; the heads side by side
-  are multiplied by a weight over all of them and by sigmoid(Wg h), and projected. n and m are state as well.
+  o = S^T q / (max(|n . q|, exp(-m')) + 1e-6). o over its own root mean square, head by head, meets a weight over all
+  heads' columns and sigmoid(Wg h), and is projected. n and m are state as well.
 
 Gates, decays, the state and o are 32-bit on every path; the projections run in the path's dtype. All projections of h
 ride in one stacked product.

@@ -16,7 +16,7 @@ experts' s divided by their sum (+ 1e-20) and multiplied by ``route_scale``.
 "softmax_groups" chooses and weighs by the softmax over all outputs of the router: s = softmax(z), the choice by
 s + correction, a group's score its largest choice score, the weights the chosen s as they are. There the last
 ``identity`` of the router's experts + identity outputs are experts without tensors that hand their input through:
-chosen, they add weight * h. Groups are formed over experts and identity experts together.
+chosen, they add weight * h. They count as neighbours of the last experts when groups are cut.
 
 Without ``gated`` an expert is Wdown_e act(Wup_e h), and so is the shared expert.
 

@@ -154,7 +154,7 @@ def test_tanh_norm_folds_a_scaled_output(dtype, size):
 
 
 MEMORY_SHAPES = [  # hidden, heads, dim, vdim
-    (64, 3, 20, 12), (48, 2, 32, 64), (50, 1, 9, 13), (96, 2, 48, 32), (64, 1, 130, 24), (32, 4, 16, 144), (40, 1, 128, 128),
+    (64, 3, 20, 12), (48, 2, 32, 80), (50, 1, 9, 13), (96, 2, 48, 64), (64, 1, 130, 24), (32, 4, 16, 144), (40, 1, 128, 128),
     (32, 2, 64, 256),
 ]
 
@@ -216,7 +216,7 @@ PIECES = ([230], [100, 2, 3, 64, 61], [180] + [1] * 50, [64, 64, 64, 38], [2] * 
 @pytest.mark.parametrize("shape", MEMORY_SHAPES)
 def test_gated_linear_attention_alone(dtype, shape):
     rt = runtime(dtype)
-    part, ref, m = gla_part(shape, dtype, rt)
+    part, ref, m = gla_part(shape, dtype, rt, rank=200 if shape[0] == 96 else 5, decay_scale=0.5 if shape[0] == 96 else 3.0)
     h = rand((230, shape[0]), 1, 1.5)
     want = memory_from_projections("gla", part, rt, ref, m, h, dtype)
     for pieces in PIECES:
@@ -241,7 +241,7 @@ def test_decays_from_nothing_kept_to_everything_kept(dtype, tau, decay_scale):
     """Decays down to e^-100 a token (what is forgotten must not come back as an overflow's NaN) and up to nearly 1 (what
     is kept over hundreds of tokens must still be there)."""
     rt = runtime(dtype)
-    shape = (64, 2, 48, 32)
+    shape = (64, 3, 48, 16)
     part, ref, m = gla_part(shape, dtype, rt, tau=tau, decay_scale=decay_scale)
     h = rand((400, shape[0]), 1, 1.5)
     want = memory_from_projections("gla", part, rt, ref, m, h, dtype)
@@ -291,7 +291,7 @@ def test_unequal_batches_against_each_alone(dtype, kind):
         part, ref, m = latent_part(LATENT_SHAPES[1], dtype, rt)
         C = LATENT_SHAPES[1][0]
     else:
-        part, ref, m = (gla_part if kind == "gla" else mlstm_part)((96, 2, 48, 32), dtype, rt)
+        part, ref, m = (gla_part if kind == "gla" else mlstm_part)((96, 2, 48, 64), dtype, rt)
         C = 96
     lengths = [150, 1, 64, 200, 65, 3]
     seqs = [rand((n, C), 40 + i, 1.2) for i, n in enumerate(lengths)]
@@ -308,6 +308,7 @@ def test_unequal_batches_against_each_alone(dtype, kind):
 LATENT_SHAPES = [  # hidden, heads, dim, rot, vdim, kv rank, q rank
     (64, 3, 16, 8, 24, 32, 40), (96, 2, 48, 16, 64, 80, 56), (50, 3, 7, 2, 5, 9, 11), (64, 5, 12, 8, 16, 32, 24),
     (96, 18, 32, 32, 16, 48, 64), (64, 1, 64, 64, 128, 112, 32), (128, 16, 128, 64, 128, 512, 96), (64, 33, 16, 16, 32, 64, 16),
+    (64, 2, 16, 8, 16, 600, 24),  # a latent wider than the tensor-core kernels take
 ]
 ROT = {"base": 500.0, "scaling": {"factor": 4.0, "original": 256, "fast": 8.0, "slow": 1.0}}
 
@@ -410,9 +411,9 @@ def test_latent_attention_finds_one_loud_key_wherever_it_sits(dtype, scaled):
 
 MOE_SHAPES = [  # hidden, experts, identity, top, ff, (groups, keep), shared ff
     (64, 5, 3, 3, 40, (4, 2), 24), (96, 7, 1, 8, 32, (1, 1), 40), (50, 3, 3, 1, 9, (1, 1), None), (50, 5, 0, 5, 11, (1, 1), 11),
-    (64, 12, 4, 2, 48, (2, 1), 64), (32, 4, 2, 2, 24, (3, 2), None), (32, 9, 0, 8, 1800, (3, 3), 8), (64, 2, 30, 4, 16, (8, 3), 16),
+    (64, 11, 3, 2, 48, (2, 1), 64), (32, 4, 2, 2, 24, (3, 2), None), (32, 9, 0, 8, 1800, (3, 3), 8), (64, 2, 30, 4, 16, (8, 3), 16),
     # rows ordered by expert and multiplied in one launch: experts with more than a tile of rows and with none
-    (96, 7, 1, 3, 72, (2, 1), 40), (256, 12, 4, 2, 64, (2, 1), 96), (136, 40, 8, 4, 264, (4, 2), None), (64, 70, 2, 2, 64, (6, 2), 8),
+    (96, 7, 1, 3, 72, (2, 1), 40), (192, 10, 5, 2, 80, (3, 1), 104), (136, 40, 8, 4, 264, (4, 2), None), (64, 70, 2, 2, 64, (6, 2), 8),
 ]
 
 

@@ -11,7 +11,7 @@ width), and one model with nothing a multiple of 4 or 8.
       | latent 5 x (12 + 8, 16) reads layer 1, q 24 + 6 experts top 2, no groups, no shared
       | mlstm 1 x (8, 72) cap 9 + dense 40
   zb  width 96, vocab 302 (sizes that tensor-core kernels take): mlstm 2 x (32, 48) cap 12 + dense 128
-      | latent 2 x (48 + 16, 64) rank 80 q 56 | gla 2 x (48, 32) rank 12 tau 3 + 7 experts and 1 identity top 8, shared 40
+      | latent 2 x (48 + 16, 64) rank 80 q 56 | gla 2 x (48, 64) rank 12 tau 3 + 7 experts and 1 identity top 8, shared 40
       | latent 4 x (16 + 16, 32) reads layer 1 + dense 96 | latent 18 x (32 + 32, 16) rank 48 (one layer's rows of its own)
       | gla 1 x (128, 112) rank 3 tau 16, mlstm 1 x (144, 80)
   zc  width 50, vocab 97 (nothing a multiple of 4 or 8): latent 3 x (7 + 2, 5) rank 9 q 11 + 3 experts and 3 identity top 1
@@ -70,7 +70,7 @@ CONFIGS = {
     "zb": {"architecture": "Zefapel", "vocab": 302, "width": 96, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "layers": _layers(
         (_memory("mlstm", 2, 32, 48, gate_cap=12.0), _dense(128)),
         (_latent(2, 48, 16, 64, 80, 56, 0.11, 5000.0, _YARN_B), None),
-        (_memory("gla", 2, 48, 32, tau=3.0), _moe(7, 1, 8, 32, None, 40)),
+        (_memory("gla", 2, 48, 64, tau=3.0), _moe(7, 1, 8, 32, None, 40)),
         (_latent(4, 16, 16, 32, 80, 24, 0.25, 5000.0, _YARN_B, kv_from=1), _dense(96)),
         (_latent(18, 32, 32, 16, 48, 64, 0.15, 300.0), None),
         (_memory("gla", 1, 128, 112, tau=16.0), None),
