@@ -7,6 +7,7 @@ from .disorax import DisoraxConfig
 from .zadunex import ZadunexConfig
 from .fogizen import FogizenConfig
 from .zefapel import ZefapelConfig
+from .givizen import GivizenConfig
 from .registry import (Architecture, architecture_name, get_architecture, known_architectures, preset_config,
                        read_config, register_architecture)
 

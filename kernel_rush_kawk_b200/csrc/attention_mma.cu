@@ -321,8 +321,12 @@ attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ qkv, i
 // read from, and outputs written into, column ranges of wider rows, the output multiplied by out_scale.
 // Options: a windowed query also sees the first keep_first keys (their pages are walked before the window's,
 // and the cache may hold them for good in its first keep_pages table entries); the output is multiplied by
-// sigmoid(gate), one number per head (mode 1) or per element (mode 2) of the row's gate columns.
+// sigmoid(gate), one number per head (mode 1) or per element (mode 2) of the row's gate columns. SHAPED: a scaled score s
+// is capped (softcap c > 0: c tanh(s / c)) and slopes[head] times the distance between query and key is taken off (slopes
+// null: nothing). tanh(t) = 1 - 2 / (1 + e^(2t)) is off by some 2^-23 of the cap, which is what a float32 score of that
+// size is off by anyway.
 // ---------------------------------------------------------------------------------
+template <bool SHAPED>
 __global__ void __launch_bounds__(THREADS)
 sink_window_prefill_kernel(bf16* __restrict__ out, int out_stride, float out_scale, const bf16* __restrict__ q_base,
                            int q_stride, int HQ, int HKV, const float* __restrict__ sink,
@@ -330,7 +334,8 @@ sink_window_prefill_kernel(bf16* __restrict__ out, int out_stride, float out_sca
                            const int* __restrict__ seq_qlen, const int* __restrict__ cu_q, const int* __restrict__ table,
                            int width, const bf16* __restrict__ k_cache, const bf16* __restrict__ v_cache,
                            float scale_log2, int window, int keep_first, int keep_pages,
-                           const bf16* __restrict__ gate, int gate_stride, int gate_mode) {
+                           const bf16* __restrict__ gate, int gate_stride, int gate_mode,
+                           const float* __restrict__ slopes, float softcap) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* smem = reinterpret_cast<bf16*>(smem_raw);  // [2 stages][K, V][64][KVP]
   const int seq = blockIdx.z, kh = blockIdx.y;
@@ -342,8 +347,10 @@ sink_window_prefill_kernel(bf16* __restrict__ out, int out_stride, float out_sca
   const int start = seq_start[seq], slot = seq_slot[seq], row0 = cu_q[seq];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int g = lane >> 2, t4 = lane & 3;
+  const float cap_log2 = softcap * LOG2E, in_cap = softcap > 0.f ? 2.f / softcap : 0.f;
 
   int pos[2], lo[2];
+  float slope[2];
   const bf16* qp[2];
   const bf16* gp[2];
   bf16* op[2];
@@ -360,6 +367,7 @@ sink_window_prefill_kernel(bf16* __restrict__ out, int out_stride, float out_sca
     op[h] = ok ? out + (size_t)(row0 + tok) * out_stride + (size_t)head * D : nullptr;
     gp[h] = (ok && gate_mode) ? gate + (size_t)(row0 + tok) * gate_stride + (gate_mode == 2 ? (size_t)head * D : (size_t)head)
                               : nullptr;
+    slope[h] = (SHAPED && slopes) ? slopes[head] * LOG2E : 0.f;
     m[h] = sink ? sink[head] * LOG2E : -INFINITY;
     l[h] = sink ? 1.f : 0.f;
   }
@@ -422,7 +430,12 @@ sink_window_prefill_kernel(bf16* __restrict__ out, int out_stride, float out_sca
       for (int c = 0; c < 4; ++c) {
         const int key = key_base + n * 8 + 2 * t4 + (c & 1);
         const int h = c >> 1;
-        s[n][c] = (whole || (key <= pos[h] && (key >= lo[h] || key < keep))) ? s[n][c] * scale_log2 : -INFINITY;
+        float x = s[n][c] * scale_log2;
+        if (SHAPED) {  // x and the cap in log2 units: e^(2 s / c) = 2^(x * 2 / c)
+          if (softcap > 0.f) x = cap_log2 * (1.f - __fdividef(2.f, 1.f + fast_exp2(x * in_cap)));
+          x -= slope[h] * (float)(pos[h] - key);
+        }
+        s[n][c] = (whole || (key <= pos[h] && (key >= lo[h] || key < keep))) ? x : -INFINITY;
       }
     softmax_update<8>(s, m, l, o);
     pv_tile_wide<8>(o, s, vs, 0, lane);
@@ -1641,13 +1654,14 @@ KRK_API int krk_attention_prefill(void* out, const void* qkv, int q_stride, int 
 }
 
 // Windowed attention with a sink for steps of many tokens. q_base and out point at the first query / output
-// column of the wider rows (strides in elements; both even, as are the column offsets).
+// column of the wider rows (strides in elements; both even, as are the column offsets). slopes (one per query head, may
+// be null) and softcap (0: none) shape the scores, see the kernel.
 KRK_API int krk_sink_window_prefill(void* out, int out_stride, float out_scale, const void* q_base, int q_stride, int HQ,
                                     int HKV, const float* sink, const int* seq_slot, const int* seq_start,
                                     const int* seq_qlen, const int* cu_q, const int* table, int width,
                                     const void* k_cache, const void* v_cache, int n_seqs, int max_q_len, float scale,
                                     int window, int keep_first, int keep_pages, const void* gate, int gate_stride,
-                                    int gate_mode, cudaStream_t stream) {
+                                    int gate_mode, const float* slopes, float softcap, cudaStream_t stream) {
   if (n_seqs == 0 || max_q_len == 0) return 0;
   const int G = HQ / HKV;
   const long long tiles = ((long long)max_q_len * G + 63) / 64;
@@ -1655,14 +1669,16 @@ KRK_API int krk_sink_window_prefill(void* out, int out_stride, float out_scale, 
   if ((out_stride & 1) || (q_stride & 1) || ((uintptr_t)out & 3) || ((uintptr_t)q_base & 3)) return -2;
   static bool configured = false;
   if (!configured) {
-    cudaFuncSetAttribute(sink_window_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)PAGE_SMEM);
+    cudaFuncSetAttribute(sink_window_prefill_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)PAGE_SMEM);
+    cudaFuncSetAttribute(sink_window_prefill_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)PAGE_SMEM);
     configured = true;
   }
   dim3 grid((unsigned)tiles, HKV, n_seqs);
-  sink_window_prefill_kernel<<<grid, THREADS, PAGE_SMEM, stream>>>(
+  auto kern = (slopes || softcap > 0.f) ? sink_window_prefill_kernel<true> : sink_window_prefill_kernel<false>;
+  kern<<<grid, THREADS, PAGE_SMEM, stream>>>(
       (bf16*)out, out_stride, out_scale, (const bf16*)q_base, q_stride, HQ, HKV, sink, seq_slot, seq_start, seq_qlen,
       cu_q, table, width, (const bf16*)k_cache, (const bf16*)v_cache, scale * LOG2E, window, keep_first, keep_pages,
-      (const bf16*)gate, gate_stride, gate_mode);
+      (const bf16*)gate, gate_stride, gate_mode, slopes, softcap);
   KRK_CHECK_LAUNCH();
   return 0;
 }

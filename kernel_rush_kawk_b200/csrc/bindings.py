@@ -52,7 +52,9 @@ _SIGNATURES = {
     "krk_lt_gemm_report": [_P, _P],
 }
 _MIX_SIGNATURES = {
-    "krk_embed_scaled": [_P, _P, _P, c_int, c_int, c_int, c_float, _P, c_int, _P, c_int],
+    "krk_embed_scaled": [_P, _P, _P, c_int, c_int, c_int, c_float, _P, c_int, _P, c_int, _P],
+    "krk_post_norm": [_P, _P, _P, _P, _P, c_float, c_int, c_int, c_float, c_int, _P],
+    "krk_tanh_cap": [_P, c_longlong, c_float, _P],
     "krk_rmsnorm_wide": [_P, _P, _P, _P, _P, c_float, c_int, c_int, c_float, _P, c_float, _P, _P, c_int, _P],
     "krk_tanh_norm": [_P, _P, _P, _P, _P, c_float, _P, _P, c_int, c_int, c_int, _P],
     "krk_gated_act": [_P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_float, c_float],
@@ -61,10 +63,11 @@ _MIX_SIGNATURES = {
     "krk_rotate_norm_write": [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, c_int, c_float, _P, _P,
                               _P, _P, c_int, _P, _P, c_int, c_int, _P, c_int, c_float, c_int, _P],
     "krk_sink_attention": [_P, c_int, c_int, c_float, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P, _P,
-                           c_int, _P, _P, c_int, c_int, c_float, c_int, c_int, c_int, _P, c_int, c_int, c_int, c_int, _P],
+                           c_int, _P, _P, c_int, c_int, c_float, c_int, c_int, c_int, _P, c_int, c_int, c_int, _P, c_float,
+                           c_int, _P],
     "krk_sink_attention_single": [_P, c_int, c_int, c_float, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P,
                                   c_int, _P, _P, c_int, c_int, c_float, c_int, c_int, _P, c_int, c_int, c_int, _P, c_int, c_int, c_float,
-                                  c_int, c_int, _P, c_int, c_int, c_int, c_int, _P],
+                                  c_int, c_int, _P, c_int, c_int, c_int, _P, c_float, c_int, _P],
     "krk_latent_norm_write": [_P, c_int, c_int, c_int, _P, c_float, _P, _P, _P, _P, c_int, c_int, _P, c_int, _P, c_int, _P],
     "krk_head_linear": [_P, c_int, c_int, c_int, c_float, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P, c_float,
                         _P, _P, c_int, c_int, _P],
@@ -73,8 +76,8 @@ _MIX_SIGNATURES = {
     "krk_latent_decode": [_P, _P, _P, c_int, c_int, c_int, c_int, _P, _P, _P, c_int, _P, c_float, c_int, c_int, _P],
     "krk_latent_gather": [_P, _P, c_int, c_int, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P],
     "krk_embed_bigram": [_P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_longlong, c_longlong, _P, _P, _P, _P, _P, c_int, _P],
-    "krk_bias_norm_rotate_write": [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_float, _P, c_int,
-                                   c_int, _P, _P, _P, _P, c_int, _P, _P, c_int, c_int, c_int, _P],
+    "krk_bias_norm_rotate_write": [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_float, c_int, c_float,
+                                   c_int, _P, c_int, c_int, _P, _P, _P, _P, c_int, _P, _P, c_int, c_int, c_int, _P],
     "krk_mixed_attention": [_P, c_int, c_int, c_float, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P, _P, _P,
                             c_int, _P, _P, c_int, c_float, c_int, _P, c_int, c_int, c_int, c_int, _P],
     "krk_mixed_attention_single": [_P, c_int, c_int, c_float, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P,
@@ -87,11 +90,11 @@ _MOE_SIGNATURES = {
     "krk_moe_route": [_P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, _P, c_int],
     "krk_moe_route_groups": [_P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P],
     "krk_moe_route_softmax_groups": [_P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P],
-    "krk_moe_gate_up_pairs": [_P, _P, c_int, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P],
+    "krk_moe_gate_up_pairs": [_P, _P, c_int, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_float, c_float, c_int, _P],
     "krk_moe_down_pairs": [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, _P, c_int, _P, c_int, _P],
     "krk_moe_sort": [_P, _P, _P, c_int, c_int, c_int, _P],
-    "krk_moe_gather": [_P, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P],
-    "krk_grouped_gemm": [_P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P, _P],
+    "krk_moe_gather": [_P, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, _P, _P, c_int, _P],
+    "krk_grouped_gemm": [_P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_float, c_float, _P, _P],
     "krk_moe_combine": [_P, _P, _P, _P, _P, _P, _P, c_int, _P, c_int, c_int, c_int, _P, c_int, _P, c_int, _P],
 }
 _MEMORY_SIGNATURES = {
@@ -128,7 +131,7 @@ _ATTN_SIGNATURES = {
     "krk_attention_prefill": [_P, _P, c_int, c_int, c_int, _P, _P, _P, _P, _P, c_int, _P, _P, c_int, c_int, c_float,
                               c_int, _P],
     "krk_sink_window_prefill": [_P, c_int, c_float, _P, c_int, c_int, c_int, _P, _P, _P, _P, _P, _P, c_int, _P, _P, c_int,
-                                c_int, c_float, c_int, c_int, c_int, _P, c_int, c_int, _P],
+                                c_int, c_float, c_int, c_int, c_int, _P, c_int, c_int, _P, c_float, _P],
     "krk_mixed_prefill": [_P, c_int, c_float, _P, c_int, c_int, c_int, _P, _P, _P, _P, _P, _P, _P, c_int, _P, _P, c_int,
                           c_int, c_float, c_int, _P, c_int, c_int, _P, c_int, _P],
     "krk_attention_decode": [_P, _P, c_int, c_int, c_int, _P, _P, _P, c_int, _P, _P, c_int, c_float, c_int, c_int, _P,
@@ -557,13 +560,42 @@ class Kernels:
             raise KernelError("a kernel input must be a 2-D tensor (or column slice) with contiguous rows")
         return t.data_ptr(), t.stride(0)
 
-    def embed_scaled(self, table, tokens, n_rows, scale, copies=1):
-        """float32 rows table[token] * scale, each written ``copies`` times side by side."""
+    def embed_scaled(self, table, tokens, n_rows, scale, copies=1, rounded=False):
+        """float32 rows table[token] * scale, each written ``copies`` times side by side. With ``rounded`` (one copy) a
+        pair: the rows, and the same rows in the table's dtype."""
+        if rounded and copies != 1:
+            raise KernelError("rounded rows come with one copy of the row")
         out = torch.empty((n_rows, copies * table.shape[1]), dtype=torch.float32, device=table.device)
+        again = torch.empty(out.shape, dtype=table.dtype, device=table.device) if rounded and table.dtype != torch.float32 else None
         self._ok(self.mix.krk_embed_scaled(out.data_ptr(), table.data_ptr(), tokens.data_ptr(), n_rows, table.shape[1],
                                            table.shape[0], float(scale), self.error.data_ptr(), _code(table.dtype),
-                                           self._stream(), int(copies)), "scaled embedding gather")
+                                           self._stream(), int(copies), _ptr(again)), "scaled embedding gather")
+        if rounded:
+            return out, (again if again is not None else out)
         return out
+
+    def post_norm(self, x, branch, gain, offset, eps, out_dtype):
+        """(x + norm(branch) * (offset + gain), the same rows in ``out_dtype``): a float32 stream takes a sublayer's output,
+        RMS-normed on its way in. Without a branch the stream is only rounded."""
+        if x.dtype != torch.float32 or not x.is_contiguous() or (branch is not None and gain.dtype != torch.float32):
+            raise KernelError("the norm of an output reads a contiguous float32 stream and a float32 gain")
+        if branch is not None and (branch.dtype != out_dtype or not branch.is_contiguous() or branch.shape != x.shape):
+            raise KernelError("a sublayer's output must have the path's dtype and the stream's shape")
+        x_new = torch.empty_like(x) if branch is not None else x
+        rows = x_new if out_dtype == torch.float32 else torch.empty(x.shape, dtype=out_dtype, device=x.device)
+        if branch is None and rows is x:
+            return x, x
+        self._ok(self.mix.krk_post_norm(x_new.data_ptr(), rows.data_ptr() if rows is not x_new else None, x.data_ptr(),
+                                        _ptr(branch), _ptr(gain), float(offset), x.shape[0], x.shape[1], float(eps),
+                                        _code(out_dtype), self._stream()), "norm of an output into the stream")
+        return x_new, rows
+
+    def tanh_cap_(self, logits, cap):
+        """logits <- cap * tanh(logits / cap), in place (float32, contiguous)."""
+        if logits.dtype != torch.float32 or not logits.is_contiguous():
+            raise KernelError("logits are capped as contiguous float32 rows")
+        self._ok(self.mix.krk_tanh_cap(logits.data_ptr(), logits.numel(), float(cap), self._stream()), "logit cap")
+        return logits
 
     def hyper_rmsnorm(self, x, branch, fold, read, gain, offset, eps, x_new, out_dtype):
         """Rows of S float32 streams side by side. With a pending ``branch``, the streams are rewritten into ``x_new``
@@ -784,10 +816,10 @@ class Kernels:
     # -- routed experts ------------------------------------------------------------------------
     MOE_PAIR_ROWS = 16  # rows up to which every (row, expert) pair reads its expert's weights by itself
 
-    def moe_route(self, x, w, b, top, gate_row=False, over_all=False, sigmoid_groups=None):
+    def moe_route(self, x, w, b, top, gate_row=False, over_all=False, sigmoid_groups=None, sigmoid=False):
         """(experts int32 [rows, top], weights float32 [rows, top], row gate float32 [rows] or None): the ``top`` largest
         of x W^T + b in 32-bit (ties: the lower index) and the softmax over them, or with ``over_all`` their shares of
-        the softmax over all experts. With ``gate_row`` the last row of W is no expert but a gate's weights: sigmoid
+        the softmax over all experts, or with ``sigmoid`` the sigmoid of each chosen logit. With ``gate_row`` the last row of W is no expert but a gate's weights: sigmoid
         of its product is the row gate. ``sigmoid_groups`` = (correction, groups, keep, scale): sigmoid scores, the choice
         by score + correction among the experts of the ``keep`` best of ``groups`` groups of neighbours, the weights
         the chosen scores over their sum, times ``scale``."""
@@ -806,7 +838,8 @@ class Kernels:
                                                    int(keep), float(scale), self._stream()), "expert routing within groups")
             return experts, weights, row_gate
         self._ok(self.moe.krk_moe_route(experts.data_ptr(), weights.data_ptr(), _ptr(row_gate), logits.data_ptr(), _ptr(b),
-                                        rows, E, int(gate_row), int(top), self._stream(), int(over_all)), "expert routing")
+                                        rows, E, int(gate_row), int(top), self._stream(), 2 if sigmoid else int(over_all)),
+                 "expert routing")
         return experts, weights, row_gate
 
     def moe_route_softmax_groups(self, x, w, correction, top, groups, keep, identity, gate_row=False):
@@ -837,24 +870,29 @@ class Kernels:
         return self.act_rows(self.linear(h, w_up), activation)
 
     def moe_experts(self, x, w_gate_up, w_down, experts, weights, intermediate, activation, add=None, add_gate=None,
-                    batch=None, gated=True, add_input=None):
+                    batch=None, gated=True, add_input=None, act_params=None, weigh_input=False):
         """add * add_gate + add_input * x + sum_j weights[r, j] * expert_{experts[r, j]}(x[r]) over the choices that are not
         -1; w_gate_up [E, 2F, K] ([E, F, K] without ``gated``), w_down [E, C, F]; ``add_gate`` (None: 1) and ``add_input``
-        (None: 0): one float32 number per row."""
+        (None: 0): one float32 number per row. ``act_params``: limit and slope of "swish_clamped". ``weigh_input``: the sum is
+        over expert(weights[r, j] * x[r]) instead."""
         rows, top = experts.shape
         E, C, F = w_down.shape
         K = x.shape[1]
         ptr, stride = self._rows_view(x)
         out = torch.empty((rows, C), dtype=x.dtype, device=x.device)
         act = _ACTIVATIONS[activation]
+        if activation == "swish_clamped" and (act_params is None or not gated):
+            raise KernelError("the clamped activation needs its limit and slope, and experts with a gate")
+        limit, slope = act_params if act_params is not None else (0.0, 1.0)
+        w_in, w_out = (weights, None) if weigh_input else (None, weights)  # which end of an expert the weights multiply
         single = batch is not None and batch.is_decode  # such a step may be replayed from a graph: nothing comes to the host
         if single or rows * top <= max(self.MOE_PAIR_ROWS * top, 2 * E):
             pairs = torch.empty((rows * top, F), dtype=x.dtype, device=x.device)
             self._ok(self.moe.krk_moe_gate_up_pairs(pairs.data_ptr(), ptr, stride, w_gate_up.data_ptr(), experts.data_ptr(),
-                                                    rows, top, F, K, act, int(gated), _code(x.dtype), self._stream()),
-                     "experts' gate/up")
+                                                    rows, top, F, K, act, int(gated), _ptr(w_in), float(limit), float(slope),
+                                                    _code(x.dtype), self._stream()), "experts' gate/up")
             self._ok(self.moe.krk_moe_down_pairs(out.data_ptr(), _ptr(add), _ptr(add_gate), pairs.data_ptr(), w_down.data_ptr(),
-                                                 experts.data_ptr(), weights.data_ptr(), rows, top, C, F, ptr, stride,
+                                                 experts.data_ptr(), _ptr(w_out), rows, top, C, F, ptr, stride,
                                                  _ptr(add_input), _code(x.dtype), self._stream()), "experts' down")
             return out
         # many rows: ordered by expert on the device; the experts' row counts come to the host (a step of many
@@ -863,9 +901,9 @@ class Kernels:
         place = torch.empty(rows * top, dtype=torch.int32, device=x.device)
         self._ok(self.moe.krk_moe_sort(offsets.data_ptr(), place.data_ptr(), experts.data_ptr(), rows, top, E,
                                        self._stream()), "expert ordering")
-        if self._use_grouped(x, K, F, C, gated):
-            return self._grouped_experts(x, w_gate_up, w_down, experts, weights, activation, add, add_gate, gated, add_input,
-                                         offsets, place)
+        if self._use_grouped(x, K, F, C, gated, activation):
+            return self._grouped_experts(x, w_gate_up, w_down, experts, w_in, w_out, activation, (limit, slope), add, add_gate,
+                                         gated, add_input, offsets, place)
         bounds = offsets.tolist()
         most = max(bounds[e + 1] - bounds[e] for e in range(E))
         cap = -(-most // 16) * 16
@@ -875,33 +913,34 @@ class Kernels:
         n_rows = E * cap if batched else rows * top
         xg = torch.empty((n_rows, K), dtype=x.dtype, device=x.device)
         self._ok(self.moe.krk_moe_gather(xg.data_ptr(), ptr, stride, place.data_ptr(), experts.data_ptr(), offsets.data_ptr(),
-                                         cap, rows, top, K, _code(x.dtype), self._stream()), "expert gather")
+                                         cap, rows, top, K, _ptr(w_in), None, _code(x.dtype), self._stream()), "expert gather")
         if batched:
             # bfloat16: every expert's rows start at a multiple of cap (the most rows any expert got), and the
             # library's batched product takes all experts at once; the rows beyond an expert's own are never read back
             gu = torch.bmm(xg.view(E, cap, K), w_gate_up.transpose(1, 2))
-            h = self.gated_act(gu.view(E * cap, 2 * F), F, activation) if gated else self.act_rows(gu.view(E * cap, F), activation)
+            h = self.gated_act(gu.view(E * cap, 2 * F), F, activation, act_params=act_params) if gated else self.act_rows(gu.view(E * cap, F), activation)
             yg = torch.bmm(h.view(E, cap, F), w_down.transpose(1, 2)).view(E * cap, C)
         else:
             yg = torch.empty((n_rows, C), dtype=x.dtype, device=x.device)
             for e in range(E):
                 a, b = bounds[e], bounds[e + 1]
                 if b > a:
-                    h = self.gate_up_act(xg[a:b], w_gate_up[e], F, activation) if gated else self.up_act(xg[a:b], w_gate_up[e], activation)
+                    h = self.gate_up_act(xg[a:b], w_gate_up[e], F, activation, act_params) if gated else self.up_act(xg[a:b], w_gate_up[e], activation)
                     yg[a:b] = self.linear(h, w_down[e])
         self._ok(self.moe.krk_moe_combine(out.data_ptr(), _ptr(add), _ptr(add_gate), yg.data_ptr(), place.data_ptr(), experts.data_ptr(),
-                                          offsets.data_ptr(), cap, weights.data_ptr(), rows, top, C, ptr, stride,
+                                          offsets.data_ptr(), cap, _ptr(w_out), rows, top, C, ptr, stride,
                                           _ptr(add_input), _code(x.dtype), self._stream()), "experts' sum")
         return out
 
     @staticmethod
-    def _use_grouped(x, K, F, C, gated) -> bool:
+    def _use_grouped(x, K, F, C, gated, activation) -> bool:
         """Whether the experts' products of many rows run as two grouped launches (sizes and alignment)."""
-        return (not gated and x.dtype == torch.bfloat16 and K % 8 == 0 and F % 8 == 0 and C % 8 == 0 and min(K, F) >= 64)
+        return ((not gated or activation == "swish_clamped") and x.dtype == torch.bfloat16 and K % 8 == 0 and F % 8 == 0 and C % 8 == 0 and min(K, F) >= 64)
 
-    def _grouped_experts(self, x, w_in, w_down, experts, weights, activation, add, add_gate, gated, add_input, offsets, place):
+    def _grouped_experts(self, x, w_first, w_down, experts, w_in, w_out, activation, act_params, add, add_gate, gated, add_input,
+                         offsets, place):
         """``moe_experts`` for many rows with the experts' row counts left on the device: rows ordered by expert, the first
-        product (the activation in its epilogue), the second, and the weighted sum."""
+        product (weights of the input and the activation in its epilogue), the second, and the weighted sum."""
         rows, top = experts.shape
         E, C, F = w_down.shape
         K = x.shape[1]
@@ -909,16 +948,17 @@ class Kernels:
         pairs = rows * top
         empty = lambda n: torch.empty((pairs, n), dtype=x.dtype, device=x.device)
         xg, h, yg = empty(K), empty(F), empty(C)
+        row_w = torch.empty(pairs, dtype=torch.float32, device=x.device) if w_in is not None else None  # in the rows' new order
         self._ok(self.moe.krk_moe_gather(xg.data_ptr(), ptr, stride, place.data_ptr(), experts.data_ptr(), offsets.data_ptr(), 0,
-                                         rows, top, K, _code(x.dtype), self._stream()), "expert gather")
-        self._ok(self.moe.krk_grouped_gemm(h.data_ptr(), xg.data_ptr(), w_in.data_ptr(), offsets.data_ptr(), pairs, E, F, K,
-                                           _ACTIVATIONS[activation], self.error.data_ptr(), self._stream()),
-                 "experts' first product")
+                                         rows, top, K, _ptr(w_in), _ptr(row_w), _code(x.dtype), self._stream()), "expert gather")
+        self._ok(self.moe.krk_grouped_gemm(h.data_ptr(), xg.data_ptr(), w_first.data_ptr(), offsets.data_ptr(), pairs, E, F, K,
+                                           _ACTIVATIONS[activation], int(gated), _ptr(row_w), float(act_params[0]),
+                                           float(act_params[1]), self.error.data_ptr(), self._stream()), "experts' first product")
         self._ok(self.moe.krk_grouped_gemm(yg.data_ptr(), h.data_ptr(), w_down.data_ptr(), offsets.data_ptr(), pairs, E, C, F, -1,
-                                           self.error.data_ptr(), self._stream()), "experts' second product")
+                                           0, None, 0.0, 0.0, self.error.data_ptr(), self._stream()), "experts' second product")
         out = torch.empty((rows, C), dtype=x.dtype, device=x.device)
         self._ok(self.moe.krk_moe_combine(out.data_ptr(), _ptr(add), _ptr(add_gate), yg.data_ptr(), place.data_ptr(),
-                                          experts.data_ptr(), offsets.data_ptr(), 0, weights.data_ptr(), rows, top, C, ptr, stride,
+                                          experts.data_ptr(), offsets.data_ptr(), 0, _ptr(w_out), rows, top, C, ptr, stride,
                                           _ptr(add_input), _code(x.dtype), self._stream()), "experts' sum")
         return out
 
@@ -968,8 +1008,9 @@ class Kernels:
                                    fuse=(k_col, v_col, inv_freq, rot_dims, value_eps))
 
     def sink_attention(self, proj, q_col, heads, dim, vdim, sink, scale, window, batch, cache, out, out_col, out_scale,
-                       fuse=None, keep_first=0, gate=None, gate_rows=None):
-        """``keep_first``: a windowed query also sees the sequence's first keys. ``gate`` (column, "head" or "element"):
+                       fuse=None, keep_first=0, gate=None, gate_rows=None, slopes=None, softcap=None):
+        """``slopes`` (float32, one per query head) and ``softcap``: a scaled score s becomes softcap * tanh(s / softcap) -
+        slope * distance, either left out where None. ``keep_first``: a windowed query also sees the sequence's first keys. ``gate`` (column, "head" or "element"):
         the result is multiplied by the sigmoid of those columns of ``gate_rows`` (default: of ``proj``)."""
         ptr, stride = self._rows_view(proj)
         optr, ostride = self._rows_view(out)
@@ -981,7 +1022,10 @@ class Kernels:
             if g_rows.dtype != proj.dtype or g_rows.shape[0] != proj.shape[0]:
                 raise KernelError("the gate's rows have the queries' dtype and number")
             (g_ptr, g_stride), g_col, g_mode = self._rows_view(g_rows), int(gate[0]), {"head": 1, "element": 2}[gate[1]]
-        extras = (keep_first, keep_pages, g_ptr, g_stride, g_col, g_mode)
+        if slopes is not None and (slopes.dtype != torch.float32 or slopes.numel() != heads):
+            raise KernelError("the distance bias takes one float32 slope per query head")
+        shape = (_ptr(slopes), float(softcap or 0.0))
+        extras = (keep_first, keep_pages, g_ptr, g_stride, g_col, g_mode, *shape)
         if batch.is_decode and proj.shape[0] == batch.n_seqs:
             # one token per sequence: a block per (sequence, kv head), its warps splitting the window's keys. The
             # choice depends on the step's shape alone, so a sequence's results do not depend on its batch
@@ -1017,7 +1061,7 @@ class Kernels:
                 _ptr(sink), batch.seq_slot.data_ptr(), batch.seq_start.data_ptr(), batch.seq_qlen.data_ptr(),
                 batch.cu_q.data_ptr(), cache.table.data_ptr(), cache.width, cache.k.data_ptr(), cache.v.data_ptr(),
                 batch.n_seqs, batch.max_q_len, float(scale), int(window or 0), keep_first, keep_pages,
-                None if g_ptr is None else g_ptr + g_col * esz, g_stride, g_mode, self._stream())
+                None if g_ptr is None else g_ptr + g_col * esz, g_stride, g_mode, *shape, self._stream())
             if rc != -2:  # -2: odd strides or offsets; the general kernel takes them
                 self._ok(rc, "tensor-core windowed attention with a sink")
                 return
@@ -1043,10 +1087,11 @@ class Kernels:
         return out
 
     def bias_norm_rotate_write(self, proj, q_col, k_col, v_col, heads, kv_heads, dim, vdim, bias, qk_gain, eps, inv_freq,
-                               rot_dims, pairs, batch, cache):
+                               rot_dims, pairs, batch, cache, unit=False, temperature=None):
         """On a stacked q | k | v product: float32 ``bias`` over all three (None: none); with ``qk_gain`` (float32, the q
         weight then the k weight, ``dim`` each) every q and k head is divided by its root mean square and multiplied by
-        it; the first ``rot_dims`` elements are rotated (``pairs``: 2i with 2i + 1, else i with i + rot_dims/2); q in
+        it (``unit``: divided only); ``temperature`` (coef, every): a q head at position p is multiplied by
+        1 + coef * ln(floor((p + 1) / every) + 1); the first ``rot_dims`` elements are rotated (``pairs``: 2i with 2i + 1, else i with i + rot_dims/2); q in
         place, k and v into their pages."""
         ptr, stride = self._rows_view(proj)
         if cache.k.dtype != proj.dtype or cache.head_dim != dim or cache.v_dim != vdim or cache.kv_heads != kv_heads:
@@ -1056,8 +1101,8 @@ class Kernels:
                 qk_gain is not None and (qk_gain.numel() != 2 * dim or qk_gain.dtype != torch.float32)):
             raise KernelError("float32 biases cover q, k and v; the float32 gains are one head's q weight and k weight")
         self._ok(self.mix.krk_bias_norm_rotate_write(
-            ptr, stride, q_col, k_col, v_col, heads, kv_heads, dim, vdim, _ptr(bias), _ptr(qk_gain), float(eps),
-            inv_freq.data_ptr(), int(rot_dims), int(bool(pairs)), batch.row_seq.data_ptr(), batch.row_pos.data_ptr(),
+            ptr, stride, q_col, k_col, v_col, heads, kv_heads, dim, vdim, _ptr(bias), _ptr(qk_gain), float(eps), int(unit),
+            float(temperature[0]) if temperature else 0.0, int(temperature[1]) if temperature else 0, inv_freq.data_ptr(), int(rot_dims), int(bool(pairs)), batch.row_seq.data_ptr(), batch.row_pos.data_ptr(),
             batch.seq_slot.data_ptr(), cache.table.data_ptr(), cache.width, cache.k.data_ptr(), cache.v.data_ptr(),
             proj.shape[0], int(getattr(cache, "keep_pages", 0)), _code(proj.dtype), self._stream()),
             "biases + head norms + rotation + cache write")

@@ -1,6 +1,8 @@
 // The routed experts' products of many rows in one launch on the 5th-generation tensor cores, the rows of an expert
 // wherever the routing put their number: C[r, :] = act(A[r, :] W_e^T) for the rows r of expert e, offsets[e] <= r <
-// offsets[e + 1], W [E, N, K]. The offsets stay on the device: the grid holds as many row tiles as the routing could need
+// offsets[e + 1], W [E, N, K]. GATED: W [E, 2N, K] holds every expert's gate rows and then its up rows; a block streams 128
+// of either, and the epilogue reads both halves of its accumulator: C = act(g, u) with g and u multiplied by the row's weight
+// first where there is one (a router that weighs an expert's input). The offsets stay on the device: the grid holds as many row tiles as the routing could need
 // at most, a block finds its expert and rows by a scan over the experts' tile counts, and blocks beyond the last tile leave
 // at once.
 //
@@ -18,10 +20,24 @@ using namespace tc;
 constexpr int BM = 128, BK = 64, UMMA_K = 16, THREADS = 192;
 constexpr uint32_t A_BYTES = BM * BK * 2;
 
-template <int BN, int STAGES>
+// act 0: silu(g) u of the two products as they would have been stored; act 3: clamped inputs,
+// g' = min(g, limit), u' = clamp(u, -limit, limit), g' sigmoid(slope g') (u' + 1), nothing rounded before the end
+__device__ __forceinline__ float gated_act_of(float g, float u, int act, float limit, float slope) {
+  if (act == 3) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.0f + expf(-slope * g)) * (u + 1.0f);
+  }
+  g = round_to<bf16>(g);
+  return g / (1.0f + expf(-g)) * round_to<bf16>(u);
+}
+
+template <int BN, int STAGES, bool GATED>
 __global__ void __launch_bounds__(THREADS)
 grouped_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w, bf16* __restrict__ C,
-                    const int* __restrict__ offsets, int E, int N, int K, int act, int* __restrict__ error) {
+                    const int* __restrict__ offsets, int E, int N, int K, int act, const float* __restrict__ row_weights,
+                    float limit, float slope, int* __restrict__ error) {
+  constexpr int BC = GATED ? BN / 2 : BN;  // columns of C a block makes
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   constexpr uint32_t B_BYTES = BN * BK * 2;
   constexpr uint32_t STAGE_BYTES = A_BYTES + B_BYTES;
@@ -56,7 +72,7 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
     before += __shfl_sync(0xffffffffu, incl, 31);
   }
   if (e < 0) return;  // the same for the whole block
-  const int n0 = blockIdx.x * BN;
+  const int n0 = blockIdx.x * BC;
   const int k_blocks = (K + BK - 1) / BK;
 
   if (threadIdx.x == 0) {
@@ -85,7 +101,8 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
       tma_load_2d(stage, &map_a, full_bar + s, kb * BK, m0);
 #pragma unroll
       for (int h = 0; h < BN / 128; ++h)
-        tma_load_2d(stage + A_BYTES + h * (128 * BK * 2), &map_w, full_bar + s, kb * BK, e * N + n0 + 128 * h);
+        tma_load_2d(stage + A_BYTES + h * (128 * BK * 2), &map_w, full_bar + s, kb * BK,
+                    GATED ? (2 * e + h) * N + n0 : e * N + n0 + 128 * h);
     }
   } else if (warp == 1 && lane == 0) {
     constexpr uint32_t idesc = umma_idesc(BM, BN);
@@ -110,10 +127,13 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
     if (!ok && lane == 0) atomicExch(error, 5);
     tc_fence_after();
     if (ok) {
+      const float a = (GATED && row_weights && row < row_end) ? row_weights[row] : 1.f;
 #pragma unroll 1
-      for (int c0 = 0; c0 < BN; c0 += 32) {
-        uint32_t g[32];
+      for (int c0 = 0; c0 < BC; c0 += 32) {
+        if (n0 + c0 >= N) break;  // the same for the whole block
+        uint32_t g[32], u[GATED ? 32 : 1];
         tmem_ld_32x32(tmem_base + ((uint32_t)(quarter * 32) << 16) + (uint32_t)c0, g);
+        if constexpr (GATED) tmem_ld_32x32(tmem_base + ((uint32_t)(quarter * 32) << 16) + (uint32_t)(BC + c0), u);
         tmem_wait_ld();
         if (row < row_end) {
           bf16* dst = C + (size_t)row * N + n0 + c0;
@@ -121,7 +141,9 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
             v[j] = __uint_as_float(g[j]);
-            if (act == 5) {  // squared relu of the product as it would have been stored
+            if constexpr (GATED) {
+              v[j] = gated_act_of(a * v[j], a * __uint_as_float(u[j]), act, limit, slope);
+            } else if (act == 5) {  // squared relu of the product as it would have been stored
               const float z = round_to<bf16>(v[j]);
               v[j] = z > 0.f ? z * z : 0.f;
             }
@@ -152,16 +174,17 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
   }
 }
 
-template <int BN, int STAGES>
-int launch_grouped(bf16* C, const bf16* A, const bf16* W, const int* offsets, int rows, int E, int N, int K, int act, int* error,
-                   cudaStream_t stream) {
+template <int BN, int STAGES, bool GATED>
+int launch_grouped(bf16* C, const bf16* A, const bf16* W, const int* offsets, int rows, int E, int N, int K, int act,
+                   const float* row_weights, float limit, float slope, int* error, cudaStream_t stream) {
+  static_assert(!GATED || BN == 256, "a gate tile and an up tile of 128 rows each");
   constexpr size_t SMEM = (size_t)STAGES * (A_BYTES + BN * BK * 2) + 1024 + (2 * STAGES + 1) * 8 + 16;
   CUtensorMap map_a, map_w;
   int rc = make_map_bf16(&map_a, A, rows, K, K, BM);
   if (rc) return rc;
-  rc = make_map_bf16(&map_w, W, (long long)E * N, K, K, 128);
+  rc = make_map_bf16(&map_w, W, (long long)E * N * (GATED ? 2 : 1), K, K, 128);
   if (rc) return rc;
-  auto kern = grouped_gemm_kernel<BN, STAGES>;
+  auto kern = grouped_gemm_kernel<BN, STAGES, GATED>;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM);
@@ -170,7 +193,9 @@ int launch_grouped(bf16* C, const bf16* A, const bf16* W, const int* offsets, in
   }
   const long long row_tiles = rows / BM + (rows < E ? rows : E);  // an expert leaves at most one tile partly filled
   if (row_tiles > 65535) return -3;
-  kern<<<dim3((N + BN - 1) / BN, (unsigned)row_tiles), THREADS, SMEM, stream>>>(map_a, map_w, C, offsets, E, N, K, act, error);
+  constexpr int BC = GATED ? BN / 2 : BN;
+  kern<<<dim3((N + BC - 1) / BC, (unsigned)row_tiles), THREADS, SMEM, stream>>>(map_a, map_w, C, offsets, E, N, K, act, row_weights,
+                                                                                limit, slope, error);
   KRK_CHECK_LAUNCH();
   return 0;
 }
@@ -178,13 +203,13 @@ int launch_grouped(bf16* C, const bf16* A, const bf16* W, const int* offsets, in
 }  // namespace
 
 // C [rows, N] = act(A [rows, K] W_e^T) over the experts' rows (offsets int32 [E + 1] on the device; rows is the most there
-// can be). act: -1 none, 5 squared relu. N and K multiples of 8, K at least 64, 16-byte aligned bases.
+// can be). act: -1 none, 5 squared relu. N and K multiples of 8, K at least 64, 16-byte aligned bases. `gated`: W [E, 2N, K],
+// act 0 (silu) or 3 (clamped swish with its limit and slope), row_weights [rows] or null.
 KRK_API int krk_grouped_gemm(void* C, const void* A, const void* W, const int* offsets, int rows, int E, int N, int K, int act,
-                             int* error, cudaStream_t stream) {
+                             int gated, const float* row_weights, float limit, float slope, int* error, cudaStream_t stream) {
   if (rows == 0 || N == 0 || E == 0) return 0;
-  if (N % 8 || K % 8 || K < 64 || (act != -1 && act != 5) || (((uintptr_t)A | (uintptr_t)W | (uintptr_t)C) & 15) ||
-      (long long)E * N > 0x7fffffffLL)
-    return -2;
-  if (N > 128) return launch_grouped<256, 4>((bf16*)C, (const bf16*)A, (const bf16*)W, offsets, rows, E, N, K, act, error, stream);
-  return launch_grouped<128, 4>((bf16*)C, (const bf16*)A, (const bf16*)W, offsets, rows, E, N, K, act, error, stream);
+  if (N % 8 || K % 8 || K < 64 || (((uintptr_t)A | (uintptr_t)W | (uintptr_t)C) & 15) || 2LL * E * N > 0x7fffffffLL) return -2;
+  if (gated ? (act != 0 && act != 3) : ((act != -1 && act != 5) || row_weights)) return -2;
+  auto go = gated ? launch_grouped<256, 4, true> : N > 128 ? launch_grouped<256, 4, false> : launch_grouped<128, 4, false>;
+  return go((bf16*)C, (const bf16*)A, (const bf16*)W, offsets, rows, E, N, K, act, row_weights, limit, slope, error, stream);
 }

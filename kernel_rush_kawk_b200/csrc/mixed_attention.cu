@@ -6,7 +6,8 @@
 // and then stores the step's last token in its place.
 //
 // krk_bias_norm_rotate_write: one warp per (row, head) of a stacked q | k | v product. Biases are added; a q or k
-// head is divided by its root mean square and multiplied by a weight of the head's size (shared by the heads); the
+// head is divided by its root mean square and (unless only the division is asked for) multiplied by a weight of the head's
+// size (shared by the heads); a q head may be multiplied by a temperature 1 + c ln(floor((p + 1) / n) + 1) of its position p; the
 // first `rot` elements are rotated by the position, element 2i with 2i + 1 (`pairs`) or i with i + rot/2; q is
 // written back in place, k and v go to their pages. All arithmetic is float32 and a value is rounded once. The
 // angle's sine and cosine are those of csrc/sink_attention.cu (frequencies as two floats each).
@@ -79,7 +80,8 @@ __global__ void embed_bigram_kernel(float* __restrict__ out, const T* __restrict
 template <typename T>
 __global__ void bias_norm_rotate_write_kernel(T* proj, int stride, int q_col, int k_col, int v_col, int HQ, int HKV, int D,
                                               int DV, const float* __restrict__ bias, const float* __restrict__ gain,
-                                              float eps, const float* __restrict__ inv_freq, int rot, int pairs,
+                                              float eps, int unit, float temp_coef, int temp_every,
+                                              const float* __restrict__ inv_freq, int rot, int pairs,
                                               const int* __restrict__ row_seq, const int* __restrict__ row_pos,
                                               const int* __restrict__ seq_slot, const int* __restrict__ table, int width,
                                               T* k_cache, T* v_cache, int rows, int keep_pages) {
@@ -124,7 +126,7 @@ __global__ void bias_norm_rotate_write_kernel(T* proj, int stride, int q_col, in
     }
   }
   float rstd = 1.f;
-  if (g) {
+  if (g || (unit && which < HQ + HKV)) {
     float sq = 0.f;
     for (int e = lane; e < n; e += 32) {
       const float x = to_float<T>(src[e]) + (b ? b[e] : 0.f);
@@ -132,6 +134,7 @@ __global__ void bias_norm_rotate_write_kernel(T* proj, int stride, int q_col, in
     }
     rstd = rsqrtf(warp_sum(sq) / (float)n + eps);
   }
+  if (temp_every > 0 && which < HQ) rstd *= 1.0f + temp_coef * logf((float)((pos + 1) / temp_every + 1));
   __syncwarp();  // q is rewritten in place: every lane has read what it needs of the head
   auto val = [&](int e) { return (to_float<T>(src[e]) + (b ? b[e] : 0.f)) * rstd * (g ? g[e] : 1.f); };
   const int half = turn >> 1;
@@ -527,8 +530,8 @@ KRK_API int krk_embed_bigram(float* out, const void* table, const void* pairs, c
 }
 
 KRK_API int krk_bias_norm_rotate_write(void* proj, int stride, int q_col, int k_col, int v_col, int HQ, int HKV, int D, int DV,
-                                       const float* bias, const float* gain, float eps, const float* inv_freq, int rot,
-                                       int pairs, const int* row_seq, const int* row_pos, const int* seq_slot,
+                                       const float* bias, const float* gain, float eps, int unit, float temp_coef,
+                                       int temp_every, const float* inv_freq, int rot, int pairs, const int* row_seq, const int* row_pos, const int* seq_slot,
                                        const int* table, int width, void* k_cache, void* v_cache, int rows, int keep_pages,
                                        int dtype, cudaStream_t stream) {
   if (rows == 0) return 0;
@@ -539,10 +542,10 @@ KRK_API int krk_bias_norm_rotate_write(void* proj, int stride, int q_col, int k_
   if (blocks > 0x7fffffffLL) return -3;
   if (dtype == KRK_DTYPE_F32)
     return (int)launch_pdl(bias_norm_rotate_write_kernel<float>, dim3((unsigned)blocks), dim3(warps * 32), 0, stream,
-                           (float*)proj, stride, q_col, k_col, v_col, HQ, HKV, D, DV, bias, gain, eps, inv_freq, rot, pairs,
+                           (float*)proj, stride, q_col, k_col, v_col, HQ, HKV, D, DV, bias, gain, eps, unit, temp_coef, temp_every, inv_freq, rot, pairs,
                            row_seq, row_pos, seq_slot, table, width, (float*)k_cache, (float*)v_cache, rows, keep_pages);
   return (int)launch_pdl(bias_norm_rotate_write_kernel<bf16>, dim3((unsigned)blocks), dim3(warps * 32), 0, stream,
-                         (bf16*)proj, stride, q_col, k_col, v_col, HQ, HKV, D, DV, bias, gain, eps, inv_freq, rot, pairs,
+                         (bf16*)proj, stride, q_col, k_col, v_col, HQ, HKV, D, DV, bias, gain, eps, unit, temp_coef, temp_every, inv_freq, rot, pairs,
                          row_seq, row_pos, seq_slot, table, width, (bf16*)k_cache, (bf16*)v_cache, rows, keep_pages);
 }
 

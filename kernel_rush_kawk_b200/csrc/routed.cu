@@ -1,8 +1,9 @@
 // Kernels of a feed-forward of routed experts.
 //
 // krk_moe_route: one warp per row. z = logits[r, :] + bias (float32); the `top` largest are taken one after
-// the other (ties: the lower index), and their weights are the softmax over the chosen logits alone, or
-// (`over_all`) each chosen expert's share of the softmax over all experts, which do not sum to one. A gate of one
+// the other (ties: the lower index), and their weights are the softmax over the chosen logits alone, or (`weigh` 1)
+// each chosen expert's share of the softmax over all experts, which do not sum to one, or (`weigh` 2) sigmoid(z) of each
+// chosen expert (sigmoid keeps the logits' order, so the choice is the same). A gate of one
 // number per row may ride in the router's product as its last column: sigmoid of it is written beside the routing and
 // multiplies what the experts' sum is added onto (a shared expert's output). (The router's product inside this
 // kernel, one block per row, was measured for single-token steps and lost to the product kernel before it: 1.72
@@ -24,7 +25,12 @@
 // and the pairs' places), krk_moe_gather copies the rows into that order, the experts' products run over
 // contiguous rows, and krk_moe_combine adds each row's weighted results onto `add`. With cap > 0 every expert's
 // rows start at a multiple of cap (expert e's i-th pair sits in row e * cap + i), which is the layout a batched
-// product over [experts, cap, K] reads.
+// batched product over [experts, cap, K] reads.
+//
+// A weight may multiply an expert's input instead of its output. The first product is linear in it: krk_moe_gate_up_pairs
+// multiplies both float32 sums by the pair's weight before anything is clamped or rounded, krk_grouped_gemm does the same in
+// its epilogue from the weights that krk_moe_gather leaves in row order, and where a library product runs in between,
+// krk_moe_gather multiplies the rows themselves. The sums of the experts' results then take no weights (null: all 1).
 #include "common.cuh"
 
 namespace {
@@ -36,16 +42,23 @@ __device__ __forceinline__ float act_of(float z, int act) {
   return 1.0f / (1.0f + expf(-z));
 }
 
+// act 3: both inputs clamped, g' = min(g, limit), u' = clamp(u, -limit, limit): g' sigmoid(slope g') (u' + 1)
+__device__ __forceinline__ float clamped_swish(float g, float u, float limit, float slope) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.0f + expf(-slope * g)) * (u + 1.0f);
+}
+
 constexpr int ROUTE_WARPS = 4;
 
 // One warp: the `top` largest of z[0..E) one after the other (z is the warp's own shared memory and is consumed),
 // their softmax weights.
 __device__ __forceinline__ void route_row(float* z, int E, int top, int lane, int* __restrict__ experts,
-                                          float* __restrict__ weights, int over_all) {
+                                          float* __restrict__ weights, int weigh) {
   float first = 0.f, total = 0.f, mine = 0.f;
   int mine_e = 0;
   float all = 0.f;
-  if (over_all) {  // the denominator over every expert, before the walk consumes z
+  if (weigh == 1) {  // the denominator over every expert, before the walk consumes z
     float big = -INFINITY;
     for (int e = lane; e < E; e += 32) big = fmaxf(big, z[e]);
     big = warp_max(big);
@@ -66,7 +79,7 @@ __device__ __forceinline__ void route_row(float* z, int E, int top, int lane, in
       if (ov > best || (ov == best && oe < best_e)) { best = ov; best_e = oe; }
     }
     if (j == 0) first = best;
-    const float p = expf(best - first);
+    const float p = weigh == 2 ? act_of(best, 2) : expf(best - first);
     total += p;
     if (lane == j) { mine = p; mine_e = best_e; }
     if (lane == 0) z[best_e] = -INFINITY;
@@ -74,7 +87,7 @@ __device__ __forceinline__ void route_row(float* z, int E, int top, int lane, in
   }
   if (lane < top) {
     experts[lane] = mine_e;
-    weights[lane] = mine / (over_all ? all : total);  // the largest logit is the first one taken
+    weights[lane] = weigh == 2 ? mine : mine / (weigh == 1 ? all : total);  // the largest logit is the first one taken
   }
 }
 
@@ -82,7 +95,7 @@ __device__ __forceinline__ void route_row(float* z, int E, int top, int lane, in
 // product), and sigmoid of it goes to row_gate
 __global__ void moe_route_kernel(int* __restrict__ experts, float* __restrict__ weights, float* __restrict__ row_gate,
                                  const float* __restrict__ logits, const float* __restrict__ bias, int rows, int E,
-                                 int has_gate, int top, int over_all) {
+                                 int has_gate, int top, int weigh) {
   extern __shared__ float z_s[];  // [warps][E]
   grid_launch_dependents();
   grid_dependency_wait();
@@ -94,7 +107,7 @@ __global__ void moe_route_kernel(int* __restrict__ experts, float* __restrict__ 
   for (int e = lane; e < E; e += 32) z[e] = src[e] + (bias ? bias[e] : 0.f);
   if (has_gate && lane == 0) row_gate[row] = act_of(src[E], 2);
   __syncwarp();
-  route_row(z, E, top, lane, experts + (size_t)row * top, weights + (size_t)row * top, over_all);
+  route_row(z, E, top, lane, experts + (size_t)row * top, weights + (size_t)row * top, weigh);
 }
 
 // The largest of z[0..n) over a warp (ties: the lower index).
@@ -213,7 +226,8 @@ constexpr int PAIR_WARPS = 8;
 template <typename T>
 __global__ void __launch_bounds__(PAIR_WARPS * 32)
 moe_gate_up_pairs_kernel(T* __restrict__ act_out, const T* __restrict__ x, int x_stride, const T* __restrict__ w,
-                         const int* __restrict__ experts, int top, int F, int K, int act, int gated) {
+                         const int* __restrict__ experts, int top, int F, int K, int act, int gated,
+                         const float* __restrict__ in_weights, float limit, float slope) {
   extern __shared__ __align__(16) float xs[];  // [K]
   grid_launch_dependents();
   grid_dependency_wait();
@@ -225,9 +239,10 @@ moe_gate_up_pairs_kernel(T* __restrict__ act_out, const T* __restrict__ x, int x
   for (int k = threadIdx.x; k < K; k += blockDim.x) xs[k] = to_float<T>(xr[k]);
   __syncthreads();
   const T* we = w + (size_t)e * (gated ? 2 : 1) * F * K;
+  const float a = in_weights ? in_weights[pair] : 1.f;
   if (!gated) {
     for (int f = blockIdx.x * PAIR_WARPS + warp; f < F; f += gridDim.x * PAIR_WARPS) {
-      const float u = warp_sum(lane_dot<T>(we + (size_t)f * K, xs, K, lane));
+      const float u = a * warp_sum(lane_dot<T>(we + (size_t)f * K, xs, K, lane));
       if (lane == 0) act_out[(size_t)pair * F + f] = from_float<T>(act_of(round_to<T>(u), act));
     }
     return;
@@ -235,8 +250,12 @@ moe_gate_up_pairs_kernel(T* __restrict__ act_out, const T* __restrict__ x, int x
   for (int f = blockIdx.x * PAIR_WARPS + warp; f < F; f += gridDim.x * PAIR_WARPS) {
     const T* wg = we + (size_t)f * K;
     const T* wu = we + (size_t)(F + f) * K;
-    const float g = warp_sum(lane_dot<T>(wg, xs, K, lane));
-    const float u = warp_sum(lane_dot<T>(wu, xs, K, lane));
+    const float g = a * warp_sum(lane_dot<T>(wg, xs, K, lane));
+    const float u = a * warp_sum(lane_dot<T>(wu, xs, K, lane));
+    if (act == 3) {
+      if (lane == 0) act_out[(size_t)pair * F + f] = from_float<T>(clamped_swish(g, u, limit, slope));
+      continue;
+    }
     // the two products leave in the path's type before the activation, as they do from a product kernel
     if (lane == 0) act_out[(size_t)pair * F + f] = from_float<T>(act_of(round_to<T>(g), act) * round_to<T>(u));
   }
@@ -310,7 +329,7 @@ moe_down_pairs_kernel(T* __restrict__ out, const T* __restrict__ add, const floa
 #pragma unroll
       for (int jj = 0; jj < 4; ++jj) {
         const float r = warp_sum(s[jj]);
-        if (on[jj]) total += weights[(size_t)row * top + j0 + jj] * round_to<T>(r);
+        if (on[jj]) total += (weights ? weights[(size_t)row * top + j0 + jj] : 1.f) * round_to<T>(r);
       }
     }
     if (lane == 0) out[(size_t)row * C + c] = from_float<T>(total);
@@ -386,13 +405,20 @@ __device__ __forceinline__ int row_of_pair(const int* __restrict__ place, const 
 
 template <typename T>
 __global__ void moe_gather_kernel(T* __restrict__ xg, const T* __restrict__ x, int x_stride, const int* __restrict__ place,
-                                  const int* __restrict__ experts, const int* __restrict__ offsets, int cap, int top, int K) {
+                                  const int* __restrict__ experts, const int* __restrict__ offsets, int cap, int top, int K,
+                                  const float* __restrict__ in_weights, float* __restrict__ row_weights) {
   grid_dependency_wait();
   const int pair = blockIdx.x;
   const T* src = x + (size_t)(pair / top) * x_stride;
   const int at = row_of_pair(place, experts, offsets, cap, pair);
   if (at < 0) return;
   T* dst = xg + (size_t)at * K;
+  if (row_weights && threadIdx.x == 0) row_weights[at] = in_weights[pair];
+  if (in_weights && !row_weights) {
+    const float a = in_weights[pair];
+    for (int k = threadIdx.x; k < K; k += blockDim.x) dst[k] = from_float<T>(a * to_float<T>(src[k]));
+    return;
+  }
   if ((K * sizeof(T)) % 16 == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0) {
     const int n = K * (int)sizeof(T) / 16;
     for (int k = threadIdx.x; k < n; k += blockDim.x) reinterpret_cast<uint4*>(dst)[k] = reinterpret_cast<const uint4*>(src)[k];
@@ -412,7 +438,7 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const T* __restrict__ ad
   const int row = blockIdx.x;
   if (threadIdx.x < top) {
     src_row[threadIdx.x] = row_of_pair(place, experts, offsets, cap, row * top + threadIdx.x);
-    src_w[threadIdx.x] = weights[(size_t)row * top + threadIdx.x];
+    src_w[threadIdx.x] = weights ? weights[(size_t)row * top + threadIdx.x] : 1.f;
   }
   __syncthreads();
   if (sizeof(T) == 2 && (C & 7) == 0 && (x_stride & 7) == 0 &&
@@ -458,13 +484,13 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const T* __restrict__ ad
 }  // namespace
 
 KRK_API int krk_moe_route(int* experts, float* weights, float* row_gate, const float* logits, const float* bias, int rows,
-                          int E, int has_gate, int top, cudaStream_t stream, int over_all) {
+                          int E, int has_gate, int top, cudaStream_t stream, int weigh) {
   if (rows == 0) return 0;
   if (top < 1 || top > 32 || top > E) return -2;
   const size_t smem = (size_t)ROUTE_WARPS * E * sizeof(float);
   if (smem > 48 * 1024) return -2;
   return (int)launch_pdl(moe_route_kernel, dim3((rows + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem, stream,
-                         experts, weights, row_gate, logits, bias, rows, E, has_gate, top, over_all);
+                         experts, weights, row_gate, logits, bias, rows, E, has_gate, top, weigh);
 }
 
 KRK_API int krk_moe_route_groups(int* experts, float* weights, float* row_gate, const float* logits, const float* correction,
@@ -497,8 +523,10 @@ KRK_API int krk_moe_route_softmax_groups(int* experts, float* weights, float* ro
 }
 
 KRK_API int krk_moe_gate_up_pairs(void* act_out, const void* x, int x_stride, const void* w, const int* experts, int rows,
-                                  int top, int F, int K, int act, int gated, int dtype, cudaStream_t stream) {
+                                  int top, int F, int K, int act, int gated, const float* in_weights, float limit, float slope,
+                                  int dtype, cudaStream_t stream) {
   if (rows == 0) return 0;
+  if (act == 3 && !gated) return -2;
   const size_t smem = (size_t)K * sizeof(float);
   if (smem > 200 * 1024 || (long long)rows * top > 65535) return -2;
   if (smem > 48 * 1024) {
@@ -508,9 +536,9 @@ KRK_API int krk_moe_gate_up_pairs(void* act_out, const void* x, int x_stride, co
   const dim3 grid((unsigned)min((F + PAIR_WARPS - 1) / PAIR_WARPS, 1024), (unsigned)(rows * top));
   if (dtype == KRK_DTYPE_F32)
     return (int)launch_pdl(moe_gate_up_pairs_kernel<float>, grid, dim3(PAIR_WARPS * 32), smem, stream, (float*)act_out,
-                           (const float*)x, x_stride, (const float*)w, experts, top, F, K, act, gated);
+                           (const float*)x, x_stride, (const float*)w, experts, top, F, K, act, gated, in_weights, limit, slope);
   return (int)launch_pdl(moe_gate_up_pairs_kernel<bf16>, grid, dim3(PAIR_WARPS * 32), smem, stream, (bf16*)act_out,
-                         (const bf16*)x, x_stride, (const bf16*)w, experts, top, F, K, act, gated);
+                         (const bf16*)x, x_stride, (const bf16*)w, experts, top, F, K, act, gated, in_weights, limit, slope);
 }
 
 KRK_API int krk_moe_down_pairs(void* out, const void* add, const float* add_gate, const void* act_in, const void* w, const int* experts,
@@ -541,15 +569,19 @@ KRK_API int krk_moe_sort(int* offsets, int* place, const int* experts, int rows,
   return (int)launch_pdl(moe_sort_kernel, dim3(1), dim3(warps * 32), smem, stream, offsets, place, experts, rows * top, E);
 }
 
+// in_weights [rows * top] (may be null): with row_weights [rows of xg] they are written there, in row order; without, the
+// rows are multiplied by them
 KRK_API int krk_moe_gather(void* xg, const void* x, int x_stride, const int* place, const int* experts, const int* offsets,
-                           int cap, int rows, int top, int K, int dtype, cudaStream_t stream) {
+                           int cap, int rows, int top, int K, const float* in_weights, float* row_weights, int dtype,
+                           cudaStream_t stream) {
   if (rows == 0) return 0;
+  if (row_weights && !in_weights) return -2;
   const int pairs = rows * top;
   if (dtype == KRK_DTYPE_F32)
     return (int)launch_pdl(moe_gather_kernel<float>, dim3(pairs), dim3(128), 0, stream, (float*)xg, (const float*)x,
-                           x_stride, place, experts, offsets, cap, top, K);
+                           x_stride, place, experts, offsets, cap, top, K, in_weights, row_weights);
   return (int)launch_pdl(moe_gather_kernel<bf16>, dim3(pairs), dim3(128), 0, stream, (bf16*)xg, (const bf16*)x, x_stride,
-                         place, experts, offsets, cap, top, K);
+                         place, experts, offsets, cap, top, K, in_weights, row_weights);
 }
 
 KRK_API int krk_moe_combine(void* out, const void* add, const float* add_gate, const void* yg, const int* place, const int* experts,

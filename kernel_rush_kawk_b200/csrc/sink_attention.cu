@@ -28,7 +28,9 @@
 // order); the result may be multiplied by sigmoid(gate), one number per head (mode 1) or per element (mode 2),
 // read from the columns `gate_col` of `gate`'s rows; the values that are written may be blended with another
 // layer's values of the same rows, (1 - lambda) v + lambda v_first. A value row of the cache may be wider than the value
-// head (`VP` elements from one to the next, DV of them read): a latent row with a rotated key part behind it.
+// head (`VP` elements from one to the next, DV of them read): a latent row with a rotated key part behind it. A scaled
+// score s may be capped (`softcap` c > 0: c tanh(s / c)), and after that `slopes[head]` times the distance from the query
+// back to the key may be taken off; the sink is a finished score and gets neither.
 #include "common.cuh"
 
 namespace {
@@ -38,6 +40,12 @@ constexpr int WIDE_V_PER_LANE = 16;  // the general kernel's second form: value 
 constexpr int WIDEST_V_PER_LANE = 32;  // its third form: up to 1,024
 
 __device__ __forceinline__ float sigmoidf_(float z) { return 1.0f / (1.0f + expf(-z)); }  // value heads up to 256
+
+// a scaled score, capped (cap > 0) and then biased by the distance between query and key
+__device__ __forceinline__ float finish_score(float s, float cap, float slope, int distance) {
+  if (cap > 0.f) s = cap * tanhf(s / cap);
+  return s - slope * (float)distance;
+}
 
 // sine and cosine of p * (f_hi + f_lo)
 __device__ __forceinline__ void angle_sincos(float p, float f_hi, float f_lo, float* s, float* c) {
@@ -146,7 +154,7 @@ __global__ void sink_attention_kernel(T* __restrict__ out, int out_stride, int o
                                       const int* __restrict__ table, int width, const T* __restrict__ k_cache,
                                       const T* __restrict__ v_cache, int VP, int rows, float scale, int window, int keep_first,
                                       int keep_pages, const T* __restrict__ gate, int gate_stride, int gate_col,
-                                      int gate_mode) {
+                                      int gate_mode, const float* __restrict__ slopes, float softcap) {
   extern __shared__ float q_s[];  // warps x D
   grid_launch_dependents();
   grid_dependency_wait();
@@ -164,6 +172,7 @@ __global__ void sink_attention_kernel(T* __restrict__ out, int out_stride, int o
   for (int d = lane; d < D; d += 32) qs[d] = to_float<T>(q[d]);
   __syncwarp();
 
+  const float slope = slopes ? slopes[head] : 0.f;
   float m = sink ? sink[head] : -INFINITY;
   float l = sink ? 1.f : 0.f;
   float acc[VPL];
@@ -181,6 +190,7 @@ __global__ void sink_attention_kernel(T* __restrict__ out, int out_stride, int o
     if (key <= hi) {
       my_page = page_of(table, width, slot, key, keep_pages);
       s = dot_row<T>(qs, k_cache + (((size_t)my_page * HKV + kh) * KRK_PAGE + (key % KRK_PAGE)) * D, D) * scale;
+      if (slopes || softcap > 0.f) s = finish_score(s, softcap, slope, pos - key);
     }
     const float m_new = fmaxf(m, warp_max(s));
     const float alpha = expf(m - m_new);  // exp(-inf) = 0 before the first key when there is no sink
@@ -257,8 +267,9 @@ sink_attention_single_kernel(T* __restrict__ out, int out_stride, int out_col, f
                              int SPL, float* __restrict__ scratch, int k_col, int v_col,
                              const float* __restrict__ inv_freq, int rot, int value_norm, float eps, T* k_cache_w,
                              T* v_cache_w, int keep_first, int keep_pages, const T* __restrict__ gate, int gate_stride,
-                             int gate_col, int gate_mode) {
+                             int gate_col, int gate_mode, const float* __restrict__ slopes, float softcap) {
   extern __shared__ __align__(16) float sm1[];
+  __shared__ float slope_s[GM];
   // a kv head's query heads are served GM at a time: blockIdx.y picks the group, all groups in one launch
   const int g0 = blockIdx.y * GM;
   const int GN = min(GM, HQ / HKV - g0);
@@ -280,6 +291,7 @@ sink_attention_single_kernel(T* __restrict__ out, int out_stride, int out_col, f
   const int first = window > 0 ? max(0, pos - window + 1) : 0;
   const T* q = proj + (size_t)seq * stride + q_col + (size_t)head0 * D;
   for (int i = threadIdx.x; i < GN * D; i += blockDim.x) q_s[i] = to_float<T>(q[i]);
+  if (threadIdx.x < GN) slope_s[threadIdx.x] = slopes ? slopes[head0 + threadIdx.x] : 0.f;
   __syncthreads();
   if (FUSE) {
     // what krk_rotate_norm_write does for this (sequence, kv head), here: the queries are rotated in shared memory,
@@ -397,7 +409,9 @@ sink_attention_single_kernel(T* __restrict__ out, int out_stride, int out_col, f
 #pragma unroll
     for (int g = 0; g < GM; ++g) {
       if (g >= GN) continue;
-      const float sc = key <= hi ? s[g] * scale : -INFINITY;
+      float sc = s[g] * scale;
+      if (slopes || softcap > 0.f) sc = finish_score(sc, softcap, slope_s[g], pos - key);
+      if (key > hi) sc = -INFINITY;
       const float m_new = fmaxf(m[g], warp_max(sc));
       const float alpha = expf(m[g] - m_new);
       p[g] = key <= hi ? expf(sc - m_new) : 0.f;
@@ -566,8 +580,8 @@ KRK_API int krk_sink_attention(void* out, int out_stride, int out_col, float out
                                int q_col, int HQ, int HKV, int D, int DV, const float* sink, const int* row_seq,
                                const int* row_pos, const int* seq_slot, const int* table, int width, const void* k_cache,
                                const void* v_cache, int v_pitch, int rows, float scale, int window, int keep_first, int keep_pages,
-                               const void* gate, int gate_stride, int gate_col, int gate_mode, int dtype,
-                               cudaStream_t stream) {
+                               const void* gate, int gate_stride, int gate_col, int gate_mode, const float* slopes,
+                               float softcap, int dtype, cudaStream_t stream) {
   if (rows == 0) return 0;
   if (DV > 32 * WIDEST_V_PER_LANE || D > 2048) return -2;
   const long long items = (long long)rows * HQ;
@@ -580,12 +594,13 @@ KRK_API int krk_sink_attention(void* out, int out_stride, int out_col, float out
     return (int)launch_pdl(widest ? sink_attention_kernel<float, WIDEST_V_PER_LANE> : wide ? sink_attention_kernel<float, WIDE_V_PER_LANE> : sink_attention_kernel<float, MAX_V_PER_LANE>, dim3((unsigned)blocks), dim3(warps * 32), smem, stream,
                            (float*)out, out_stride, out_col, out_scale, (const float*)proj, stride, q_col, HQ, HKV, D, DV,
                            sink, row_seq, row_pos, seq_slot, table, width, (const float*)k_cache, (const float*)v_cache,
-                           v_pitch, rows, scale, window, keep_first, keep_pages, (const float*)gate, gate_stride, gate_col, gate_mode);
+                           v_pitch, rows, scale, window, keep_first, keep_pages, (const float*)gate, gate_stride, gate_col, gate_mode,
+                           slopes, softcap);
   return (int)launch_pdl(widest ? sink_attention_kernel<bf16, WIDEST_V_PER_LANE> : wide ? sink_attention_kernel<bf16, WIDE_V_PER_LANE> : sink_attention_kernel<bf16, MAX_V_PER_LANE>,
                          dim3((unsigned)blocks), dim3(warps * 32), smem, stream, (bf16*)out,
                          out_stride, out_col, out_scale, (const bf16*)proj, stride, q_col, HQ, HKV, D, DV, sink, row_seq,
                          row_pos, seq_slot, table, width, (const bf16*)k_cache, (const bf16*)v_cache, v_pitch, rows, scale, window,
-                         keep_first, keep_pages, (const bf16*)gate, gate_stride, gate_col, gate_mode);
+                         keep_first, keep_pages, (const bf16*)gate, gate_stride, gate_col, gate_mode, slopes, softcap);
 }
 
 // One token per sequence: rows are the sequences, in order. Value heads of up to 512 elements; others take
@@ -599,7 +614,8 @@ KRK_API int krk_sink_attention_single(void* out, int out_stride, int out_col, fl
                                       const void* v_cache, int v_pitch, int n_seqs, float scale, int window, int splits,
                                       float* scratch, int fuse, int k_col, int v_col, const float* inv_freq, int rot,
                                       int value_norm, float eps, int keep_first, int keep_pages, const void* gate,
-                                      int gate_stride, int gate_col, int gate_mode, int dtype, cudaStream_t stream) {
+                                      int gate_stride, int gate_col, int gate_mode, const float* slopes, float softcap,
+                                      int dtype, cudaStream_t stream) {
   if (n_seqs == 0) return 0;
   if (DV > 512 || D > 1024) return -2;
   const int G = HQ / HKV;
@@ -627,7 +643,7 @@ KRK_API int krk_sink_attention_single(void* out, int out_stride, int out_col, fl
                      (float*)out, out_stride, out_col, out_scale, (const float*)proj, stride, q_col, HQ, HKV, D, DV, sink,
                      seq_slot, seq_start, table, width, (const float*)k_cache, (const float*)v_cache, v_pitch, scale, window, SPL, scratch, k_col, v_col,
                      inv_freq, rot, value_norm, eps, (float*)k_cache, (float*)v_cache, keep_first, keep_pages,
-                     (const float*)gate, gate_stride, gate_col, gate_mode);
+                     (const float*)gate, gate_stride, gate_col, gate_mode, slopes, softcap);
     } else {
       auto kern = wide ? (v4 ? sink_attention_single_kernel<bf16, true, false, 16, 4> : sink_attention_single_kernel<bf16, false, false, 16, 4>)
                   : fuse ? (v4 ? sink_attention_single_kernel<bf16, true, true, 4, GROUP_MAX> : sink_attention_single_kernel<bf16, false, true, 4, GROUP_MAX>)
@@ -637,7 +653,7 @@ KRK_API int krk_sink_attention_single(void* out, int out_stride, int out_col, fl
                      (bf16*)out, out_stride, out_col, out_scale, (const bf16*)proj, stride, q_col, HQ, HKV, D, DV, sink,
                      seq_slot, seq_start, table, width, (const bf16*)k_cache, (const bf16*)v_cache, v_pitch, scale, window, SPL, scratch, k_col, v_col,
                      inv_freq, rot, value_norm, eps, (bf16*)k_cache, (bf16*)v_cache, keep_first, keep_pages,
-                     (const bf16*)gate, gate_stride, gate_col, gate_mode);
+                     (const bf16*)gate, gate_stride, gate_col, gate_mode, slopes, softcap);
     }
     if (e != cudaSuccess) return (int)e;
   }

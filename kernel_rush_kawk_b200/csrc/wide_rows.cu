@@ -8,6 +8,13 @@
 // second result from the same pass. The gains are float32. One block per row, the row
 // held in shared memory, global memory read once.
 //
+// krk_post_norm: the norm of a sublayer's output on its way into the stream. s = x + (y * rsqrt(mean(y^2) + eps)) *
+// (offset + w), y the output in the path's type; s goes back as the float32 stream and, rounded, as the rows that the next
+// sublayer reads. Without an output it only rounds the stream. A thread keeps its pieces of both rows in registers, so that
+// the stream's are on their way while the output's sum of squares is formed.
+//
+// krk_tanh_cap: z <- c tanh(z / c) in place over float32 rows (logits).
+//
 // krk_tanh_norm stands in a norm's place without being one: s = x + f * branch with an optional vector f (float32),
 // y = tanh(alpha * s) * w + b, element by element.
 #include "common.cuh"
@@ -16,7 +23,7 @@ namespace {
 
 template <typename T>
 __global__ void embed_scaled_kernel(float* __restrict__ out, const T* __restrict__ table, const int* __restrict__ ids,
-                                    int H, int n_table_rows, float scale, int* error, int copies) {
+                                    int H, int n_table_rows, float scale, int* error, int copies, T* __restrict__ rounded) {
   grid_launch_dependents();
   grid_dependency_wait();
   const int r = blockIdx.x;
@@ -28,6 +35,7 @@ __global__ void embed_scaled_kernel(float* __restrict__ out, const T* __restrict
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
     const float v = bad ? 0.f : to_float<T>(src[i]) * scale;
     for (int c = 0; c < copies; ++c) dst[(size_t)c * H + i] = v;
+    if (rounded) rounded[(size_t)r * H + i] = from_float<T>(v);  // the same row as the first sublayer reads it
   }
 }
 
@@ -119,6 +127,92 @@ __global__ void rmsnorm_wide_kernel(T* __restrict__ out, float* x_new, const flo
   }
 }
 
+constexpr int POST_ITEMS = 4;  // pieces of four elements that a thread keeps
+
+// VEC: H a multiple of 4 and at most 4 * POST_ITEMS * blockDim.x. Otherwise element by element, rows read twice.
+template <typename T, bool VEC>
+__global__ void post_norm_kernel(float* __restrict__ x_new, T* __restrict__ rows, const float* __restrict__ x,
+                                 const T* __restrict__ y, const float* __restrict__ gain, float offset, int H, float eps) {
+  __shared__ float scratch[32];
+  grid_launch_dependents();
+  const size_t base = (size_t)blockIdx.x * H;
+  if (VEC) {
+    float4 w[POST_ITEMS], f[POST_ITEMS];
+    float b[POST_ITEMS][4];
+    if (y) {
+#pragma unroll
+      for (int k = 0; k < POST_ITEMS; ++k) {
+        const int i = threadIdx.x + k * blockDim.x;
+        if (4 * i < H) w[k] = reinterpret_cast<const float4*>(gain)[i];
+      }
+    }
+    grid_dependency_wait();
+    float sq = 0.f;
+    if (y) {
+#pragma unroll
+      for (int k = 0; k < POST_ITEMS; ++k) {
+        const int i = threadIdx.x + k * blockDim.x;
+        if (4 * i < H) load4_rows<T>(y + base + 4 * i, b[k]);
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < POST_ITEMS; ++k) {
+      const int i = threadIdx.x + k * blockDim.x;
+      if (4 * i < H) f[k] = reinterpret_cast<const float4*>(x + base)[i];
+    }
+    if (y) {
+#pragma unroll
+      for (int k = 0; k < POST_ITEMS; ++k)
+        if (4 * (int)(threadIdx.x + k * blockDim.x) < H) sq += b[k][0] * b[k][0] + b[k][1] * b[k][1] + b[k][2] * b[k][2] + b[k][3] * b[k][3];
+    }
+    const float rstd = y ? rsqrtf(block_sum(sq, scratch) / (float)H + eps) : 0.f;
+#pragma unroll
+    for (int k = 0; k < POST_ITEMS; ++k) {
+      const int i = threadIdx.x + k * blockDim.x;
+      if (4 * i >= H) continue;
+      float r[4] = {f[k].x, f[k].y, f[k].z, f[k].w};
+      if (y) {
+        r[0] += b[k][0] * rstd * (offset + w[k].x);
+        r[1] += b[k][1] * rstd * (offset + w[k].y);
+        r[2] += b[k][2] * rstd * (offset + w[k].z);
+        r[3] += b[k][3] * rstd * (offset + w[k].w);
+        store4_rows<float>(x_new + base + 4 * i, r);
+      }
+      if (rows) store4_rows<T>(rows + base + 4 * i, r);
+    }
+    return;
+  }
+  grid_dependency_wait();
+  float sq = 0.f;
+  if (y)
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+      const float b = to_float<T>(y[base + i]);
+      sq += b * b;
+    }
+  const float rstd = y ? rsqrtf(block_sum(sq, scratch) / (float)H + eps) : 0.f;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    float r = x[base + i];
+    if (y) {
+      r += to_float<T>(y[base + i]) * rstd * (offset + gain[i]);
+      x_new[base + i] = r;
+    }
+    if (rows) rows[base + i] = from_float<T>(r);
+  }
+}
+
+__global__ void tanh_cap_kernel(float* __restrict__ z, long long n, float cap) {
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const long long i = 4 * ((long long)blockIdx.x * blockDim.x + threadIdx.x);
+  if (i + 4 <= n) {
+    float4 v = *reinterpret_cast<float4*>(z + i);
+    v.x = cap * tanhf(v.x / cap); v.y = cap * tanhf(v.y / cap); v.z = cap * tanhf(v.z / cap); v.w = cap * tanhf(v.w / cap);
+    *reinterpret_cast<float4*>(z + i) = v;
+  } else {
+    for (long long j = i; j < n; ++j) z[j] = cap * tanhf(z[j] / cap);
+  }
+}
+
 // V elements a thread (four where sizes and addresses allow); blockIdx.y walks the row
 template <typename T, bool VEC>
 __global__ void tanh_norm_kernel(T* __restrict__ out, float* x_new, const float* x, const T* __restrict__ branch,
@@ -199,14 +293,14 @@ __global__ void gated_act_kernel(T* __restrict__ out, const T* __restrict__ gu, 
 }  // namespace
 
 KRK_API int krk_embed_scaled(float* out, const void* table, const int* ids, int rows, int H, int n_table_rows, float scale,
-                             int* error, int dtype, cudaStream_t stream, int copies) {
+                             int* error, int dtype, cudaStream_t stream, int copies, void* rounded) {
   if (rows == 0) return 0;
   if (copies < 1) return -2;
   if (dtype == KRK_DTYPE_F32)
     return (int)launch_pdl(embed_scaled_kernel<float>, dim3(rows), dim3(128), 0, stream, out, (const float*)table, ids, H,
-                           n_table_rows, scale, error, copies);
+                           n_table_rows, scale, error, copies, (float*)rounded);
   return (int)launch_pdl(embed_scaled_kernel<bf16>, dim3(rows), dim3(128), 0, stream, out, (const bf16*)table, ids, H,
-                         n_table_rows, scale, error, copies);
+                         n_table_rows, scale, error, copies, (bf16*)rounded);
 }
 
 template <typename T>
@@ -231,6 +325,36 @@ KRK_API int krk_rmsnorm_wide(void* out, float* x_new, const float* x, const void
   return dtype == KRK_DTYPE_F32
              ? launch_rmsnorm_wide<float>(out, x_new, x, branch, gain, offset, rows, H, eps, branch2, bscale, gain2, out2, stream)
              : launch_rmsnorm_wide<bf16>(out, x_new, x, branch, gain, offset, rows, H, eps, branch2, bscale, gain2, out2, stream);
+}
+
+template <typename T>
+static int launch_post_norm(float* x_new, void* rows_out, const float* x, const void* y, const float* gain, float offset,
+                            int rows, int H, float eps, cudaStream_t stream) {
+  int threads = 32;
+  while (threads < 1024 && 4 * POST_ITEMS * threads < H) threads <<= 1;
+  while (threads < 256 && 4 * threads < H) threads <<= 1;  // up to 256 threads: fewer pieces each
+  const bool vec = H % 4 == 0 && H <= 4 * POST_ITEMS * threads && ((uintptr_t)gain & 15) == 0;
+  auto kern = vec ? post_norm_kernel<T, true> : post_norm_kernel<T, false>;
+  return (int)launch_pdl(kern, dim3(rows), dim3(threads), 0, stream, x_new, (T*)rows_out, x, (const T*)y, gain, offset, H, eps);
+}
+
+// y (the path's type, may be null: then x is only rounded into `rows` and gain and x_new are not looked at); `rows` may be
+// null where nobody reads the rounded rows
+KRK_API int krk_post_norm(float* x_new, void* rows_out, const float* x, const void* y, const float* gain, float offset, int rows,
+                          int H, float eps, int dtype, cudaStream_t stream) {
+  if (rows == 0) return 0;
+  if (y && (!gain || !x_new)) return -2;
+  return dtype == KRK_DTYPE_F32 ? launch_post_norm<float>(x_new, rows_out, x, y, gain, offset, rows, H, eps, stream)
+                                : launch_post_norm<bf16>(x_new, rows_out, x, y, gain, offset, rows, H, eps, stream);
+}
+
+// n floats from a 16-byte aligned address
+KRK_API int krk_tanh_cap(float* z, long long n, float cap, cudaStream_t stream) {
+  if (n == 0) return 0;
+  if (!(cap > 0.f) || ((uintptr_t)z & 15)) return -2;
+  const long long blocks = (n + 1023) / 1024;
+  if (blocks > 0x7fffffffLL) return -3;
+  return (int)launch_pdl(tanh_cap_kernel, dim3((unsigned)blocks), dim3(256), 0, stream, z, n, cap);
 }
 
 template <typename T>

@@ -162,7 +162,7 @@ class Model:
             x = self.embedding.forward(ctx)
         if self.position is not None:
             x = self.position.on_embeddings(ctx, x)
-        stream = Stream(x)
+        stream = x if isinstance(x, Stream) else Stream(x)
         ctx.shared = {}  # what a layer leaves for later layers of the same step (values that they blend in, say)
         for run, entry in enumerate(self.plan.schedule):
             stream = self.blocks[entry.layer].forward(ctx, stream, ctx.cache_view(run))

@@ -9,7 +9,7 @@ from .norm import Normed, RMSNorm
 from .rope import RotaryTable
 from .attention import GQAttention
 from .mlp import SwiGLU
-from .block import ParallelResidualBlock, PreNormBlock
+from .block import OutputNormBlock, ParallelResidualBlock, PreNormBlock
 from .embedding import BigramEmbedding, OutputHead, TokenEmbedding
 from .wide import DenseMLP, GatedMLP, ScaledEmbedding, WideRMSNorm
 from .branches import Branch, ParallelMixer

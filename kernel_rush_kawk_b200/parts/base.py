@@ -100,7 +100,7 @@ class Embedding(Part):
         return None
 
     def forward(self, ctx):
-        """The step's rows [rows, hidden] from ``ctx.batch.tokens``."""
+        """The step's rows [rows, hidden] from ``ctx.batch.tokens``, or a ``Stream`` that starts from them."""
         raise NotImplementedError
 
 
@@ -169,16 +169,20 @@ class Stream:
 
     With hyper-connections ``x`` holds several streams side by side and ``fold`` the
     weights with which the pending output is written back into them (parts/hyper.py); a
-    norm that scales outputs element by element leaves that vector there (parts/tanh_norm.py)."""
+    norm that scales outputs element by element leaves that vector there (parts/tanh_norm.py).
 
-    __slots__ = ("x", "branch", "branch2", "scale", "fold")
+    Where sublayers read the stream itself (norms on their outputs only), ``rows`` holds x as they read it, in the path's
+    dtype; whoever changes x writes it anew or clears it."""
 
-    def __init__(self, x, branch=None, branch2=None, scale=1.0, fold=None):
+    __slots__ = ("x", "branch", "branch2", "scale", "fold", "rows")
+
+    def __init__(self, x, branch=None, branch2=None, scale=1.0, fold=None, rows=None):
         self.x = x
         self.branch = branch
         self.branch2 = branch2
         self.scale = scale
         self.fold = fold
+        self.rows = rows
 
 
 # ----------------------------------------------------------------------------

@@ -8,6 +8,10 @@ stay pending with their multiplier and the next norm folds them in, in 32-bit.
 (engine/model.py:294-302 of willzeng274/kernel-rush-kawk). The adds are not done
 here: a branch output stays pending on the stream and the next norm, wherever it
 sits (this layer, the next one, or the final norm), folds it in.
+
+"output_norm" has its norms on the sublayers' outputs only: x <- x + norm1(Mixer(x)); x <- x + norm2(FeedForward(x)).
+The sublayers read x itself, rounded to the path's dtype; the kernel that norms an output adds it to the stream and
+leaves the rounded rows of the new x for the sublayer after it, so nothing stays pending.
 """
 
 from __future__ import annotations
@@ -59,5 +63,21 @@ class ParallelResidualBlock(Block):
         return stream
 
 
+class OutputNormBlock(Block):
+    def __init__(self, mixer_norm, mixer, feed_forward_norm, feed_forward):
+        super().__init__(mixer_norm, mixer, feed_forward_norm, feed_forward)
+        if not all(hasattr(n, "fold_output") for n in (mixer_norm, feed_forward_norm) if n is not None):
+            raise TypeError("norms on outputs need a norm that folds an output into the stream (rmsnorm_wide)")
+
+    def forward(self, ctx, stream: Stream, cache) -> Stream:
+        y = self.mixer.forward(ctx, self.mixer_norm.read_stream(ctx, stream), cache)
+        self.mixer_norm.fold_output(ctx, stream, y)
+        if self.feed_forward is not None:
+            y = self.feed_forward.forward(ctx, self.feed_forward_norm.read_stream(ctx, stream))
+            self.feed_forward_norm.fold_output(ctx, stream, y)
+        return stream
+
+
 register_block("prenorm", PreNormBlock)
+register_block("output_norm", OutputNormBlock)
 register_block("parallel_residual", ParallelResidualBlock)

@@ -58,14 +58,16 @@ class BigramEmbedding(Embedding):
 
 
 class OutputHead(Head):
-    """params: vocab, hidden, scale (default 1: the logits are multiplied by it). The plan points
-    "weight" at the embedding table's checkpoint name when the head is tied."""
+    """params: vocab, hidden, scale (default 1: the logits are multiplied by it), softcap (default None; c: the logits
+    become c * tanh(logits / c), after the scale). The plan points "weight" at the embedding table's checkpoint
+    name when the head is tied."""
 
     def __init__(self, params):
         super().__init__(params)
         self.vocab = int(params["vocab"])
         self.hidden = int(params["hidden"])
         self.scale = float(params.get("scale", 1.0))
+        self.softcap = None if params.get("softcap") is None else float(params["softcap"])
         self.weight = None
 
     def tensor_specs(self):
@@ -77,7 +79,9 @@ class OutputHead(Head):
     def forward(self, ctx, h):
         """h: normalised rows (a Normed or a tensor) of the wanted positions."""
         logits = ctx.ops.linear(h, self.weight, out_float32=True)
-        return logits if self.scale == 1.0 else logits.mul_(self.scale)
+        if self.scale != 1.0:
+            logits.mul_(self.scale)
+        return logits if self.softcap is None else ctx.ops.tanh_cap_(logits, self.softcap)
 
 
 register_embedding("token_embedding", TokenEmbedding)

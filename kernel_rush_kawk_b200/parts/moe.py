@@ -18,6 +18,12 @@ s + correction, a group's score its largest choice score, the weights the chosen
 ``identity`` of the router's experts + identity outputs are experts without tensors that hand their input through:
 chosen, they add weight * h. They count as neighbours of the last experts when groups are cut.
 
+"sigmoid" chooses by the logits and weighs by their sigmoid as it is, without a correction and without renormalising.
+
+``weigh_input``: a token's weight for an expert multiplies the expert's input, not its output: the result is the sum of
+expert_e(w_e h). The activation "swish_clamped" clamps both products at ``limit`` (the shared expert's at
+``shared_limit``) and has a ``slope``, see parts/wide.py.
+
 Without ``gated`` an expert is Wdown_e act(Wup_e h), and so is the shared expert.
 
 The routing never leaves the device: a routing kernel writes each row's experts and
@@ -43,7 +49,8 @@ class RoutedExperts(FeedForward):
     has a bias "router.b"), weights ("chosen", the default: softmax over the chosen logits; "all": each chosen
     expert's share of the softmax over all experts, not renormalised), scoring (None, "sigmoid_groups" with
     groups, keep_groups and route_scale, or "softmax_groups" with groups, keep_groups and identity; both have the tensor
-    "correction" and no router bias), gated (default True: experts have a gate product)."""
+    "correction" and no router bias; or "sigmoid", which has neither), gated (default True: experts have a gate product),
+    weigh_input (default False), limit, slope (default 1.702) and shared_limit (default: limit) of "swish_clamped"."""
 
     def __init__(self, params):
         super().__init__(params)
@@ -58,8 +65,15 @@ class RoutedExperts(FeedForward):
         self.router_bias = bool(p.get("router_bias", True))
         self.weights = str(p.get("weights", "chosen"))
         self.scoring = p.get("scoring")
-        if self.scoring not in (None, "sigmoid_groups", "softmax_groups"):
-            raise ValueError(f"scoring must be None, 'sigmoid_groups' or 'softmax_groups', got {self.scoring!r}")
+        if self.scoring not in (None, "sigmoid", "sigmoid_groups", "softmax_groups"):
+            raise ValueError(f"scoring must be None, 'sigmoid', 'sigmoid_groups' or 'softmax_groups', got {self.scoring!r}")
+        self.grouped = self.scoring in ("sigmoid_groups", "softmax_groups")  # a correction, and groups of neighbours
+        self.weigh_input = bool(p.get("weigh_input", False))
+        self.act_params = self.shared_act_params = None
+        if self.activation == "swish_clamped":
+            slope = float(p.get("slope", 1.702))
+            self.act_params = (float(p["limit"]), slope)
+            self.shared_act_params = (float(p["limit"] if p.get("shared_limit") is None else p["shared_limit"]), slope)
         self.gated = bool(p.get("gated", True))
         self.identity = int(p.get("identity", 0))
         if self.identity and self.scoring != "softmax_groups":
@@ -70,6 +84,7 @@ class RoutedExperts(FeedForward):
         self.route_scale = float(p.get("route_scale", 1.0))
         if self.scoring:
             self.router_bias = False
+        if self.grouped:
             if outputs % self.groups or not 1 <= self.keep_groups <= self.groups:
                 raise ValueError(f"{outputs} experts do not form {self.groups} equal groups of which {self.keep_groups} are kept")
             if self.top > self.keep_groups * (outputs // self.groups):
@@ -86,7 +101,7 @@ class RoutedExperts(FeedForward):
         specs = {"router": TensorSpec((self.outputs, H))}
         if self.router_bias:
             specs["router.b"] = TensorSpec((self.experts,), "vector")
-        if self.scoring:
+        if self.grouped:
             specs["correction"] = TensorSpec((self.outputs,), "vector")
         for e in range(self.experts):
             if self.gated:
@@ -107,7 +122,7 @@ class RoutedExperts(FeedForward):
         # in the path's dtype: the logits' product accumulates in 32-bit; the shared expert's gate is its last row
         self.router_w = torch.cat([tensors["router"]] + ([tensors["shared.sg"]] if self.shared_gate else []), dim=0).contiguous()
         self.router_b = tensors["router.b"].float().contiguous() if self.router_bias else None
-        self.correction = tensors["correction"].float().contiguous() if self.scoring else None
+        self.correction = tensors["correction"].float().contiguous() if self.grouped else None
         first = ("gate", "up") if self.gated else ("up",)  # what is stacked into an expert's first product
         self.w_gate_up = torch.stack([torch.cat([tensors[f"e{e}.{k}"] for k in first], dim=0) for e in range(E)]).contiguous()
         self.w_down = torch.stack([tensors[f"e{e}.down"] for e in range(E)]).contiguous()
@@ -121,7 +136,8 @@ class RoutedExperts(FeedForward):
         x = h.tensor() if hasattr(h, "tensor") and not isinstance(h, torch.Tensor) else h
         base = None
         if self.shared is not None:
-            act = (ops.gate_up_act(x, self.w_shared_in, self.shared, self.activation) if self.gated
+            shaped = {} if self.shared_act_params is None else {"act_params": self.shared_act_params}
+            act = (ops.gate_up_act(x, self.w_shared_in, self.shared, self.activation, **shaped) if self.gated
                    else ops.up_act(x, self.w_shared_in, self.activation))
             base = ops.linear(act, self.w_shared_down)
         if self.scoring == "softmax_groups":
@@ -130,7 +146,9 @@ class RoutedExperts(FeedForward):
                                                                               gate_row=self.shared_gate)
             return ops.moe_experts(x, self.w_gate_up, self.w_down, experts, weights, self.intermediate, self.activation,
                                    add=base, add_gate=row_gate, batch=ctx.batch, gated=self.gated, add_input=passed)
-        if self.scoring:
+        if self.scoring == "sigmoid":
+            experts, weights, row_gate = ops.moe_route(x, self.router_w, None, self.top, gate_row=self.shared_gate, sigmoid=True)
+        elif self.scoring:
             experts, weights, row_gate = ops.moe_route(x, self.router_w, None, self.top, gate_row=self.shared_gate,
                                                        sigmoid_groups=(self.correction, self.groups, self.keep_groups,
                                                                        self.route_scale))
@@ -139,8 +157,13 @@ class RoutedExperts(FeedForward):
                                                        over_all=True)
         else:
             experts, weights, row_gate = ops.moe_route(x, self.router_w, self.router_b, self.top, gate_row=self.shared_gate)
+        options = {} if self.gated else {"gated": False}
+        if self.act_params is not None:
+            options["act_params"] = self.act_params
+        if self.weigh_input:
+            options["weigh_input"] = True
         return ops.moe_experts(x, self.w_gate_up, self.w_down, experts, weights, self.intermediate, self.activation,
-                               add=base, add_gate=row_gate, batch=ctx.batch, **({} if self.gated else {"gated": False}))
+                               add=base, add_gate=row_gate, batch=ctx.batch, **options)
 
 
 register_feed_forward("routed_experts", RoutedExperts)

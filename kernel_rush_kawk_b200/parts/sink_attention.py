@@ -33,6 +33,14 @@ pairs element 2i with element 2i + 1 instead of i with i + rot_dims/2. ``rot_fac
 divided by it. ``chunk``: a query at position p sees the keys of its own block of ``chunk`` positions only,
 (p // chunk) * chunk .. p, blocks counted from the sequence's first position. ``talk``: the heads' scaled scores of
 a (query, key) pair are mixed before the softmax, s'_h = sum_g T[h, g] s_g with a learned T ("talk", [heads, heads]).
+
+Options of the scores, which the windowed kernels take as they are. ``softcap`` c: a scaled score s becomes c tanh(s / c).
+``distance_bias``: after that slope_h * (i - j) is taken off the score of query position i and key position j, with
+slope_h = 2^(-8 (h + 1) / heads) for head h = 0 .. heads - 1; the sink's term gets neither. ``q_temp`` (coef, every): a q
+head at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1), after its norm; ``qk_norm`` "head_rms": q and
+k heads are divided by their root mean square without a weight. A windowed layer, or one with one of these options, with
+per-head norms or a temperature runs the row kernel of the second kind (norms, temperature, cache write in one pass) and
+then the windowed attention kernels.
 """
 
 from __future__ import annotations
@@ -46,8 +54,9 @@ from .branches import Branch
 class SinkWindowAttention(Branch):
     """params: hidden, heads, kv_heads, dim, vdim, scale, window (None or int), rot_dims, rot_base,
     value_norm (bool), sink (bool), eps, keep_first (int), gate (None, "head" or "element"),
-    value_mix (None, "first" or "blend"), value_mix_key, bias (bool), qk_norm (None, "row" or "head"); sink may
-    be "zero"; rot_pairs (bool), rot_factor, chunk (None or int), talk (bool)."""
+    value_mix (None, "first" or "blend"), value_mix_key, bias (bool), qk_norm (None, "row", "head" or "head_rms"); sink
+    may be "zero"; rot_pairs (bool), rot_factor, chunk (None or int), talk (bool); softcap (None or a number),
+    distance_bias (bool), q_temp (None or (coef, every))."""
 
     def __init__(self, params):
         super().__init__(params)
@@ -66,14 +75,24 @@ class SinkWindowAttention(Branch):
         self.has_sink = bool(p.get("sink", False)) and not self.zero_sink
         self.bias = bool(p.get("bias", False))
         self.qk_norm = p.get("qk_norm")
-        if self.qk_norm not in (None, "row", "head"):
-            raise ValueError(f"qk_norm must be None, 'row' or 'head', got {self.qk_norm!r}")
+        if self.qk_norm not in (None, "row", "head", "head_rms"):
+            raise ValueError(f"qk_norm must be None, 'row', 'head' or 'head_rms', got {self.qk_norm!r}")
         self.rot_pairs = bool(p.get("rot_pairs", False))
         self.rot_factor = float(p.get("rot_factor", 1.0))
         self.chunk = None if p.get("chunk") is None else int(p["chunk"])
         self.talk = bool(p.get("talk", False))
-        #: the second kind of this attention (see the module text)
-        self._mixed = self.qk_norm == "head" or self.rot_pairs or self.chunk is not None or self.talk
+        self.softcap = None if p.get("softcap") is None else float(p["softcap"])
+        self.distance_bias = bool(p.get("distance_bias", False))
+        self.q_temp = None if p.get("q_temp") is None else (float(p["q_temp"][0]), int(p["q_temp"][1]))
+        if self.softcap is not None and not self.softcap > 0:
+            raise ValueError(f"softcap must be positive, got {self.softcap}")
+        if self.q_temp is not None and self.q_temp[1] < 1:
+            raise ValueError(f"q_temp's second number must be at least 1, got {self.q_temp[1]}")
+        #: the row kernel of the second kind (see the module text): per-head norms, pair rotation, temperature
+        self._row_pass = self.qk_norm in ("head", "head_rms") or self.rot_pairs or self.q_temp is not None
+        shaped = self.window is not None or self.softcap is not None or self.distance_bias
+        #: the attention kernel of the second kind
+        self._mixed = self.chunk is not None or self.talk or (self._row_pass and not shaped)
         self.eps = float(p.get("eps", 0.0))
         self.keep_first = int(p.get("keep_first") or 0) if self.window is not None else 0
         self.gate = p.get("gate")
@@ -87,10 +106,11 @@ class SinkWindowAttention(Branch):
             raise ValueError(f"heads ({self.heads}) must be a multiple of kv_heads ({self.kv_heads})")
         if self.rot_dims % 2 or self.rot_dims > self.dim:
             raise ValueError(f"rot_dims ({self.rot_dims}) must be even and at most dim ({self.dim})")
-        if self._mixed and (self.window is not None or self.value_norm or self.value_mix or self.qk_norm == "row"
-                            or self.gate == "element" or (self.chunk is not None and self.chunk < 1)):
-            raise ValueError("per-head norms, pair rotation, blocks of keys and mixed scores come without a window, value "
-                             "norm, value blend, row norm or per-element gate")
+        if self._mixed and (shaped or self.gate == "element" or (self.chunk is not None and self.chunk < 1)):
+            raise ValueError("blocks of keys and mixed scores come without a window, score cap, distance bias or per-element gate")
+        if (self._mixed or self._row_pass) and (self.value_norm or self.value_mix or self.qk_norm == "row"):
+            raise ValueError("per-head norms, pair rotation, temperatures, blocks of keys and mixed scores come without a "
+                             "value norm, value blend or row norm")
 
     def tensor_specs(self):
         specs = {"q": TensorSpec((self.heads * self.dim, self.hidden)),
@@ -122,11 +142,9 @@ class SinkWindowAttention(Branch):
 
     @property
     def _plain(self) -> bool:
-        return not (self.keep_first or self.gate or self.value_mix)
+        return not (self.keep_first or self.gate or self.value_mix or self.distance_bias or self.softcap)
 
     def attention_head_dims(self):
-        if self._mixed:
-            return (self.dim,) if self.dim == self.vdim and self.dim % 16 == 0 and self.dim <= 256 else ()
         """Steps of many tokens in bfloat16 run on the tensor cores where key and value heads have one size that
         is a multiple of 16: that kernel is compiled per head size."""
         return (self.dim,) if self.dim == self.vdim and self.dim % 16 == 0 and self.dim <= 256 else ()
@@ -137,9 +155,13 @@ class SinkWindowAttention(Branch):
         self.sink = tensors["sink"].float().contiguous() if self.has_sink else None
         if self.zero_sink:
             self.sink = torch.zeros(self.heads, dtype=torch.float32, device=runtime.device)
+        self.slopes = None
+        if self.distance_bias:  # in 64-bit on the host, rounded once
+            self.slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / self.heads) for h in range(self.heads)], dtype=torch.float64)
+            self.slopes = self.slopes.to(torch.float32).to(runtime.device)
         f = lambda *keys: torch.cat([tensors[k].float().reshape(-1) for k in keys]).contiguous()
         self.qkv_bias = f("q.b", "k.b", "v.b") if self.bias else None
-        self.qk_gain = f("q.norm", "k.norm") if self.qk_norm else None
+        self.qk_gain = f("q.norm", "k.norm") if self.qk_norm in ("row", "head") else None
         # the few rotation frequencies come from the host in 64-bit, so that they depend on no device's pow()
         # and as two floats each (the float32 value, then what float32 leaves of the float64 value)
         i = torch.arange(self.rot_dims // 2, dtype=torch.float64)
@@ -160,12 +182,25 @@ class SinkWindowAttention(Branch):
         k_col = self.heads * self.dim
         v_col = k_col + self.kv_heads * self.dim
         value_eps = self.eps if self.value_norm else None
-        if self._mixed:
+        gate = (v_col + self.kv_heads * self.vdim, self.gate) if self.gate else None
+        shape = {}
+        if self.distance_bias or self.softcap is not None:
+            shape = {"slopes": self.slopes, "softcap": self.softcap}
+        if self._mixed or self._row_pass:
+            more = {}
+            if self.qk_norm == "head_rms":
+                more["unit"] = True
+            if self.q_temp is not None:
+                more["temperature"] = self.q_temp
             ops.bias_norm_rotate_write(proj, 0, k_col, v_col, self.heads, self.kv_heads, self.dim, self.vdim, self.qkv_bias,
-                                       self.qk_gain, self.eps, self.inv_freq, self.rot_dims, self.rot_pairs, ctx.batch, cache)
-            gate = (v_col + self.kv_heads * self.vdim, self.gate) if self.gate else None
-            ops.mixed_attention(proj, 0, self.heads, self.dim, self.vdim, self.sink, self.talk_w, self.scale, self.chunk,
-                                ctx.batch, cache, out, col0, scale, gate=gate)
+                                       self.qk_gain, self.eps, self.inv_freq, self.rot_dims, self.rot_pairs, ctx.batch, cache,
+                                       **more)
+            if self._mixed:
+                ops.mixed_attention(proj, 0, self.heads, self.dim, self.vdim, self.sink, self.talk_w, self.scale, self.chunk,
+                                    ctx.batch, cache, out, col0, scale, gate=gate)
+            else:
+                ops.sink_attention(proj, 0, self.heads, self.dim, self.vdim, self.sink, self.scale, self.window, ctx.batch,
+                                   cache, out, col0, scale, keep_first=self.keep_first, gate=gate, **shape)
             return
         if self.bias or self.qk_norm:  # biases onto q, k, v; q and k rows divided by their root mean square
             ops.bias_row_norm(proj, (0, k_col, v_col, v_col + self.kv_heads * self.vdim), self.qkv_bias, self.qk_gain,
@@ -182,9 +217,8 @@ class SinkWindowAttention(Branch):
                 blend = (first, self.lam)
             ops.rotate_norm_write(proj, 0, k_col, v_col, self.heads, self.kv_heads, self.dim, self.vdim, self.inv_freq,
                                   self.rot_dims, value_eps, ctx.batch, cache, value_mix=blend)
-            gate = (v_col + self.kv_heads * self.vdim, self.gate) if self.gate else None
             ops.sink_attention(proj, 0, self.heads, self.dim, self.vdim, self.sink, self.scale, self.window, ctx.batch,
-                               cache, out, col0, scale, keep_first=self.keep_first, gate=gate)
+                               cache, out, col0, scale, keep_first=self.keep_first, gate=gate, **shape)
             return
         if ctx.batch.is_decode and ops.sink_attention_step(proj, 0, k_col, v_col, self.heads, self.kv_heads, self.dim,
                                                            self.vdim, self.inv_freq, self.rot_dims, value_eps, self.sink,

@@ -7,7 +7,8 @@
   gain. The stream it leaves behind (``x_new``) is float32. A stream with two
   pending outputs and a multiplier is folded as x + scale * (branch + branch2);
   ``forward_pair`` gives two norms of the same x (two gains, one pass over x) for
-  a layer whose mixer and feed-forward both read it.
+  a layer whose mixer and feed-forward both read it. ``fold_output`` norms a sublayer's
+  output instead, on its way into the stream: x <- x + y / sqrt(mean(y^2) + eps) * (offset + w).
 * ``GatedMLP``: down(act(gate h) * (up h)) with the activation as a parameter
   (``gelu_tanh``: 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))), or ``silu``);
   the activation and the product are computed in float32 and rounded once.
@@ -30,7 +31,8 @@ ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "sigmoid": 2}
 
 class ScaledEmbedding(Embedding):
     """params: vocab, hidden, scale, copies (default 1: the row is written that many times side by side, the
-    equal streams that hyper-connections start from)."""
+    equal streams that hyper-connections start from), rounded (default False: the rows are also left in the path's
+    dtype, for sublayers that read the stream itself)."""
 
     def __init__(self, params):
         super().__init__(params)
@@ -38,6 +40,9 @@ class ScaledEmbedding(Embedding):
         self.hidden = int(params["hidden"])
         self.scale = float(params.get("scale", 1.0))
         self.copies = int(params.get("copies", 1))
+        self.rounded = bool(params.get("rounded", False))
+        if self.rounded and self.copies != 1:
+            raise ValueError("rounded rows come with one copy of the stream")
         self.table = None
 
     def tensor_specs(self):
@@ -47,6 +52,9 @@ class ScaledEmbedding(Embedding):
         self.table = tensors["table"]
 
     def forward(self, ctx):
+        if self.rounded:
+            x, rows = ctx.ops.embed_scaled(self.table, ctx.batch.tokens, ctx.batch.n_rows, self.scale, rounded=True)
+            return Stream(x, rows=rows)
         if self.copies == 1:
             return ctx.ops.embed_scaled(self.table, ctx.batch.tokens, ctx.batch.n_rows, self.scale)
         return ctx.ops.embed_scaled(self.table, ctx.batch.tokens, ctx.batch.n_rows, self.scale, copies=self.copies)
@@ -79,6 +87,18 @@ class WideRMSNorm(Norm):
             raise ValueError("two norms of one x share their size, eps and gain offset")
         return self._run(ctx, stream, other.gain)
 
+    def fold_output(self, ctx, stream: Stream, y) -> None:
+        """This norm of a sublayer's output ``y`` is added to the stream; ``stream.rows`` is left up to date."""
+        if stream.branch is not None or stream.branch2 is not None:
+            raise TypeError("an output that is normed on its way into the stream finds no other one pending")
+        stream.x, stream.rows = ctx.ops.post_norm(stream.x, y, self.gain, self.offset, self.eps, self.dtype)
+
+    def read_stream(self, ctx, stream: Stream):
+        """The stream itself as a sublayer reads it, in the path's dtype (no norm)."""
+        if stream.rows is None:
+            stream.rows = ctx.ops.post_norm(stream.x, None, None, 0.0, 0.0, self.dtype)[1]
+        return stream.rows
+
     def _run(self, ctx, stream: Stream, gain2):
         x = stream.x
         if x.dtype != torch.float32:
@@ -98,6 +118,7 @@ class WideRMSNorm(Norm):
             normed.mark_fused(r)  # computed here and now: a product never folds this norm into its prologue
             out.append(normed)
         stream.x = x_new
+        stream.rows = None
         stream.branch = stream.branch2 = None
         stream.scale = 1.0
         return out

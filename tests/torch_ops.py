@@ -183,7 +183,19 @@ def _act(z, name):
 
 
 class _WideOps:
-    def embed_scaled(self, table, tokens, n_rows, scale, copies=1):
+    def post_norm(self, x, branch, gain, offset, eps, out_dtype):
+        if branch is not None:
+            y = branch.float()
+            x = x + y * torch.rsqrt((y * y).mean(dim=-1, keepdim=True) + eps) * (offset + gain.float())
+        return x, x.to(out_dtype)
+
+    def tanh_cap_(self, logits, cap):
+        return logits.copy_(cap * torch.tanh(logits / cap))
+
+    def embed_scaled(self, table, tokens, n_rows, scale, copies=1, rounded=False):
+        if rounded:
+            x = table[tokens.long()].float() * scale
+            return x, x.to(self.dtype)
         return (table[tokens.long()].float() * scale).repeat(1, copies)
 
     def rmsnorm_wide(self, x, branch, gain, offset, eps, x_new, out_dtype, branch2=None, scale=1.0, gain2=None):
@@ -230,7 +242,7 @@ class _WideOps:
         out[:, out_col:out_col + heads * n] = y.to(out.dtype)
         return out
 
-    def moe_route(self, x, w, b, top, gate_row=False, over_all=False, sigmoid_groups=None):
+    def moe_route(self, x, w, b, top, gate_row=False, over_all=False, sigmoid_groups=None, sigmoid=False):
         z = x.float() @ w.float().t()
         row_gate = torch.sigmoid(z[:, -1]) if gate_row else None
         z = z[:, :-1] if gate_row else z
@@ -239,6 +251,8 @@ class _WideOps:
         if b is not None:
             z = z + b.float()
         best = torch.topk(z, top, dim=-1)  # ties are not exercised: equal logits do not occur with random weights
+        if sigmoid:
+            return best.indices.to(torch.int32), torch.sigmoid(best.values), row_gate
         if over_all:
             return best.indices.to(torch.int32), torch.softmax(z, dim=-1).gather(1, best.indices), row_gate
         return best.indices.to(torch.int32), torch.softmax(best.values, dim=-1), row_gate
@@ -261,7 +275,7 @@ class _WideOps:
         return table[tok].float() + pairs[row].float()
 
     def bias_norm_rotate_write(self, proj, q_col, k_col, v_col, heads, kv_heads, dim, vdim, bias, qk_gain, eps, inv_freq,
-                               rot_dims, pairs, batch, cache):
+                               rot_dims, pairs, batch, cache, unit=False, temperature=None):
         rows = proj.shape[0]
         pos = batch.row_pos.long()
         half = rot_dims // 2
@@ -275,6 +289,12 @@ class _WideOps:
         if qk_gain is not None:
             q = q * torch.rsqrt((q * q).mean(dim=-1, keepdim=True) + eps) * qk_gain[:dim]
             k = k * torch.rsqrt((k * k).mean(dim=-1, keepdim=True) + eps) * qk_gain[dim:]
+        elif unit:
+            q = q * torch.rsqrt((q * q).mean(dim=-1, keepdim=True) + eps)
+            k = k * torch.rsqrt((k * k).mean(dim=-1, keepdim=True) + eps)
+        if temperature is not None:
+            coef, every = temperature
+            q = q * (1.0 + coef * torch.log(((pos + 1) // every + 1).float()))[:, None, None]
 
         def rotate(t):
             if not half:
@@ -429,7 +449,7 @@ class _WideOps:
         out[:, out_col:out_col + inner] = (v.reshape(rows, inner) * weight * out_scale).to(out.dtype)
 
     def moe_experts(self, x, w_gate_up, w_down, experts, weights, intermediate, activation, add=None, add_gate=None,
-                    batch=None, gated=True, add_input=None):
+                    batch=None, gated=True, add_input=None, act_params=None, weigh_input=False):
         rows, top = experts.shape
         out = torch.zeros((rows, w_down.shape[1]), dtype=torch.float32) if add is None else add.float().clone()
         if add is not None and add_gate is not None:
@@ -442,10 +462,13 @@ class _WideOps:
                 e = int(experts[r, j])
                 if e < 0:
                     continue
-                gu = xf[r] @ w_gate_up[e].float().t()
-                a = _act(gu[:intermediate], activation)
-                a = (a * gu[intermediate:] if gated else a).to(self.dtype).float()
-                out[r] += weights[r, j] * (a @ w_down[e].float().t())
+                gu = xf[r] @ w_gate_up[e].float().t() * (weights[r, j] if weigh_input else 1.0)
+                if activation == "swish_clamped":
+                    a = self.gated_act(gu[None], intermediate, activation, act_params=act_params)[0]
+                else:
+                    a = _act(gu[:intermediate], activation)
+                    a = a * gu[intermediate:] if gated else a
+                out[r] += (1.0 if weigh_input else weights[r, j]) * (a.to(self.dtype).float() @ w_down[e].float().t())
         return out.to(self.dtype)
 
     def rotate_norm_write(self, proj, q_col, k_col, v_col, heads, kv_heads, dim, vdim, inv_freq, rot_dims, value_eps,
@@ -479,7 +502,7 @@ class _WideOps:
         cache.v[page, :, pos % PAGE] = v.to(proj.dtype)
 
     def sink_attention(self, proj, q_col, heads, dim, vdim, sink, scale, window, batch, cache, out, out_col, out_scale,
-                       keep_first=0, gate=None, gate_rows=None):
+                       keep_first=0, gate=None, gate_rows=None, slopes=None, softcap=None):
         rows = proj.shape[0]
         G = heads // cache.kv_heads
         q = proj[:, q_col:q_col + heads * dim].reshape(rows, heads, dim).float()
@@ -501,6 +524,10 @@ class _WideOps:
                 visible &= (positions[None, :] > qpos[:, None] - window) | (positions[None, :] < keep_first)
             for h in range(heads):
                 s = (q[row0:row0 + n, h] @ k[:, h // G].t()) * scale
+                if softcap:
+                    s = softcap * torch.tanh(s / softcap)
+                if slopes is not None:
+                    s = s - slopes[h] * (qpos[:, None] - positions[None, :]).float()
                 s = s.masked_fill(~visible, float("-inf"))
                 m = s.max(dim=-1, keepdim=True).values
                 extra = 0.0
