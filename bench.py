@@ -50,6 +50,11 @@ width and heads (attention over cached low-rank rows, routed experts with a shar
 Zadunex decoder of about that size (the other model whose matrix states outweigh its attention), and beside the Qwen3
 decoder of that size.
 
+``--only design_givizen`` measures the Givizen decoder (windowed attention with capped scores, distance biases, per-head
+norms and query temperatures, norms on the sublayers' outputs, routed experts whose weights multiply their inputs and a
+shared one) at two sizes beside its closest existing model, the Disorax decoder of equal width, heads and experts, and
+beside the Qwen3 decoder of that size.
+
 ``--only workload_8b`` and ``--only workload_14b`` run the baseline's two larger
 configurations (Qwen3-8B sizes: 8 prompts of 256 to 2,048 tokens, 128 greedy steps;
 Qwen3-14B sizes: 16 prompts of 512 to 4,096 tokens, 128 steps at temperature 0.7)
@@ -233,6 +238,10 @@ DESIGN_SIZES = {
                       "head_dim": 128, "vocab_size": 32768},
     "zefapel_lite": {"hidden_size": 2048, "intermediate_size": 8192, "num_attention_heads": 16, "num_key_value_heads": 4,
                      "head_dim": 128, "vocab_size": 32768},
+    "givizen_small": {"hidden_size": 1024, "intermediate_size": 2048, "num_attention_heads": 8, "num_key_value_heads": 2,
+                      "head_dim": 128, "vocab_size": 32768},
+    "givizen_lite": {"hidden_size": 2048, "intermediate_size": 11264, "num_attention_heads": 16, "num_key_value_heads": 4,
+                     "head_dim": 128, "vocab_size": 32768},
     "fogizen_1b": {"hidden_size": 1536, "intermediate_size": 6144, "num_attention_heads": 12, "num_key_value_heads": 4,
                    "head_dim": 128, "vocab_size": 32768},
     "fogizen_4b": {"hidden_size": 2560, "intermediate_size": 9728, "num_attention_heads": 32, "num_key_value_heads": 8,
@@ -241,11 +250,12 @@ DESIGN_SIZES = {
 #: a design's closest existing model of equal size, measured beside it as well (preset -> presets)
 DESIGN_NEIGHBOURS = {"zadunex_1b": ("taredra_1b",), "zadunex_4b": ("taredra_4b",), "fogizen_1b": ("taredra_1b",),
                      "fogizen_4b": ("taredra_4b",), "zefapel_small": ("disorax_small", "zadunex_1b"),
-                     "zefapel_lite": ("disorax_lite", "zadunex_4b")}
+                     "zefapel_lite": ("disorax_lite", "zadunex_4b"), "givizen_small": ("disorax_small",),
+                     "givizen_lite": ("disorax_lite",)}
 KERNEL_FAMILIES = {
     "product": ("_skinny", "_library_gemm", "_gemm_nt", "gemm_tcgen05"),
-    "norm": ("rmsnorm", "add_rmsnorm", "rmsnorm_wide", "hyper_rmsnorm", "norm_sum", "tanh_norm"),
-    "activation": ("swiglu", "gated_act", "act_rows"),
+    "norm": ("rmsnorm", "add_rmsnorm", "rmsnorm_wide", "hyper_rmsnorm", "norm_sum", "tanh_norm", "post_norm"),
+    "activation": ("swiglu", "gated_act", "act_rows", "tanh_cap_"),
     "attention": ("rope_attention", "rotate_norm_write", "sink_attention", "latent_norm_write", "head_linear",
                   "bias_row_norm", "bias_norm_rotate_write", "mixed_attention", "latent_rows", "rotated_latent_attention"),
     "recurrence": ("token_shift", "linear_recurrence", "causal_conv_silu", "ssd_scan", "gated_group_norm", "gla_scan",
@@ -678,7 +688,7 @@ def main() -> int:
     p.add_argument("--impl", default="ours", choices=["ours", "reference"])
     p.add_argument("--only", default="", choices=["", "prefill", "decode_b1", "decode_b8", "decode_b16", "decode_b32", "decode_b64",
                                                   "workload_8b", "workload_14b", "design_taredra", "design_disorax",
-                                                  "design_zadunex", "design_fogizen", "design_zefapel"],
+                                                  "design_zadunex", "design_fogizen", "design_zefapel", "design_givizen"],
                    help="run one piece only (for profiling), or one of the baseline's larger configurations end to end")
     p.add_argument("--layers", type=int, default=0, help="run fewer layers than the model has (both numbers are reported)")
     args = p.parse_args()

@@ -54,6 +54,8 @@ __device__ __forceinline__ int page_off(int key, int piece) {
 }
 constexpr float LOG2E = 1.4426950408889634f;
 
+constexpr size_t PAGE_SMEM = (size_t)2 * 2 * TILE_ELEMS * sizeof(bf16);  // two stages of a page of keys and one of values
+
 // Copy one page [64][D] of one kv head to shared memory [64][DP], all threads of the block.
 __device__ __forceinline__ void load_page(bf16* dst, const bf16* __restrict__ src) {
   constexpr int CHUNKS = KRK_PAGE * (D / 8);
@@ -454,6 +456,166 @@ sink_window_prefill_kernel(bf16* __restrict__ out, int out_stride, float out_sca
         b /= 1.0f + expf(-__bfloat162float(gp[h][n * 8 + 2 * t4 + 1]));
       }
       *reinterpret_cast<uint32_t*>(op[h] + n * 8 + 2 * t4) = pack_bf16x2(a, b);
+    }
+  }
+}
+
+// ---------------------------------------------------------------------------------
+// The same attention for a single token of every sequence. Block = (key split, kv head x row tile of 16 query heads,
+// sequence), the splits of an item a thread-block cluster; a block brings every `splits`-th page that its query sees to
+// shared memory (kept first pages before the window's), warp w works on keys 16 w .. 16 w + 15 of each with running
+// statistics of its own. The warps' shares meet in shared memory, the blocks' in the first block's, through distributed
+// shared memory, both in a fixed order; the sink enters once, as the first warp's starting state in the first block.
+// ---------------------------------------------------------------------------------
+__global__ void __launch_bounds__(THREADS)
+sink_window_decode_kernel(bf16* __restrict__ out, int out_stride, float out_scale, const bf16* __restrict__ q_base,
+                          int q_stride, int HQ, int HKV, const float* __restrict__ sink, const int* __restrict__ seq_slot,
+                          const int* __restrict__ seq_start, const int* __restrict__ table, int width,
+                          const bf16* __restrict__ k_cache, const bf16* __restrict__ v_cache, float scale_log2, int window,
+                          int keep_first, int keep_pages, const bf16* __restrict__ gate, int gate_stride, int gate_mode,
+                          const float* __restrict__ slopes, float softcap, int row_tiles, int inbox_rows) {
+  namespace cg = cooperative_groups;
+  cg::cluster_group cluster = cg::this_cluster();
+  asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");  // "I have started"
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  bf16* smem = reinterpret_cast<bf16*>(smem_raw);                     // [2 stages][K, V][64][KVP]
+  float* inbox = reinterpret_cast<float*>(smem_raw + PAGE_SMEM);      // [splits][inbox_rows][D + 2], the first block's is used
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int split = blockIdx.x, n_splits = gridDim.x;
+  const int kh = blockIdx.y / row_tiles, rt = blockIdx.y % row_tiles;
+  const int seq = blockIdx.z;
+  const int G = HQ / HKV;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int g = lane >> 2, t4 = lane & 3;
+  const int pos = seq_start[seq], slot = seq_slot[seq];  // the new token sits at `pos`, its key is cached
+  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  const int keep = window > 0 ? keep_first : 0;
+  const int j_first = lo / KRK_PAGE;
+  const int n_kept = keep > 0 ? min((keep - 1) / KRK_PAGE + 1, j_first) : 0;
+  const int n_steps = n_kept + pos / KRK_PAGE - j_first + 1;
+  const int ring = max(width - keep_pages, 1);
+  const size_t page_stride = (size_t)HKV * KRK_PAGE * D, head_off = (size_t)kh * KRK_PAGE * D;
+  auto page_index = [&](int i) { return i < n_kept ? i : j_first + (i - n_kept); };
+  auto issue = [&](int i, int stage) {
+    const int j = page_index(i);
+    const int page = table[(size_t)slot * width + (j < keep_pages ? j : keep_pages + (j - keep_pages) % ring)];
+    bf16* ks = smem + (size_t)stage * 2 * TILE_ELEMS;
+    load_page(ks, k_cache + (size_t)page * page_stride + head_off);
+    load_page(ks + TILE_ELEMS, v_cache + (size_t)page * page_stride + head_off);
+    cp_async_commit();
+  };
+  if (split < n_steps) issue(split, 0);
+
+  const float cap_log2 = softcap * LOG2E, in_cap = softcap > 0.f ? 2.f / softcap : 0.f;
+  const bf16* qp[2];
+  float m[2], l[2], slope[2];
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    const int r = rt * 16 + g + 8 * h;
+    const int head = kh * G + r;
+    qp[h] = r < G ? q_base + (size_t)seq * q_stride + (size_t)head * D : nullptr;
+    slope[h] = (slopes && r < G) ? slopes[head] * LOG2E : 0.f;
+    const bool has = sink && split == 0 && warp == 0 && r < G;
+    m[h] = has ? sink[head] * LOG2E : -INFINITY;
+    l[h] = has ? 1.f : 0.f;
+  }
+  uint32_t qf[KSTEPS][4];
+  load_q(qf, qp[0], qp[1], lane);
+  float o[DTILES][4];
+#pragma unroll
+  for (int n = 0; n < DTILES; ++n)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) o[n][c] = 0.f;
+
+  int stage = 0;
+  for (int i = split; i < n_steps; i += n_splits, stage ^= 1) {
+    if (i + n_splits < n_steps) {
+      issue(i + n_splits, stage ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    const bf16* ks = smem + (size_t)stage * 2 * TILE_ELEMS;
+    const int key0 = warp * 16, base = page_index(i) * KRK_PAGE + key0;
+    float s[2][4];
+    qk_tile<2>(s, qf, ks, key0, lane);
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        const int key = base + n * 8 + 2 * t4 + (c & 1), h = c >> 1;
+        float x = s[n][c] * scale_log2;
+        if (softcap > 0.f) x = cap_log2 * (1.f - __fdividef(2.f, 1.f + fast_exp2(x * in_cap)));  // as in the prompt kernel
+        x -= slope[h] * (float)(pos - key);
+        s[n][c] = (key <= pos && (key >= lo || key < keep)) ? x : -INFINITY;
+      }
+    softmax_update<2>(s, m, l, o);
+    pv_tile_wide<2>(o, s, ks + TILE_ELEMS, key0, lane);
+    __syncthreads();
+  }
+
+  constexpr int RP = D + 2;
+  float* red = reinterpret_cast<float*>(smem_raw);  // [4 warps][16 rows][RP]; the page buffers are free now
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    float* dst = red + ((size_t)warp * 16 + g + 8 * h) * RP;
+    if (t4 == 0) { dst[D] = m[h]; dst[D + 1] = l[h]; }
+#pragma unroll
+    for (int n = 0; n < DTILES; ++n)
+      *reinterpret_cast<float2*>(dst + n * 8 + 2 * t4) = make_float2(o[n][2 * h], o[n][2 * h + 1]);
+  }
+  __syncthreads();
+  asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");  // every block of the cluster has started
+  const int rows = min(16, G - rt * 16);
+  float* inbox0 = cluster.map_shared_rank(inbox, 0);
+  for (int r = warp; r < rows; r += 4) {
+    float mw[4], big = -INFINITY;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) { mw[w] = red[((size_t)w * 16 + r) * RP + D]; big = fmaxf(big, mw[w]); }
+    const float safe = big == -INFINITY ? 0.f : big;
+    float wgt[4], lsum = 0.f;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) { wgt[w] = exp2f(mw[w] - safe); lsum += wgt[w] * red[((size_t)w * 16 + r) * RP + D + 1]; }
+    float* dst = inbox0 + ((size_t)split * inbox_rows + r) * RP;
+    for (int d = lane; d < D; d += 32) {
+      float acc = 0.f;
+#pragma unroll
+      for (int w = 0; w < 4; ++w) acc += wgt[w] * red[((size_t)w * 16 + r) * RP + d];
+      dst[d] = acc;
+    }
+    if (lane == 0) { dst[D] = big; dst[D + 1] = lsum; }
+  }
+  cluster.sync();  // every block's share has arrived in the first block
+  if (split != 0) return;
+  for (int r = warp; r < rows; r += 4) {
+    const float* mine = inbox + (size_t)r * RP;
+    const size_t step = (size_t)inbox_rows * RP;
+    const int head = kh * G + rt * 16 + r;
+    float big = -INFINITY;
+    for (int sp = 0; sp < n_splits; ++sp) big = fmaxf(big, mine[sp * step + D]);
+    float lsum = 0.f, acc[(D + 31) / 32];
+#pragma unroll
+    for (int i = 0; i < (D + 31) / 32; ++i) acc[i] = 0.f;
+    for (int sp = 0; sp < n_splits; ++sp) {
+      const float w = exp2f(mine[sp * step + D] - big);
+      lsum += w * mine[sp * step + D + 1];
+#pragma unroll
+      for (int i = 0; i < (D + 31) / 32; ++i)
+        if (lane + 32 * i < D) acc[i] += w * mine[sp * step + lane + 32 * i];
+    }
+    float inv = out_scale / lsum;
+    const bf16* gp = gate_mode ? gate + (size_t)seq * gate_stride : nullptr;
+    if (gate_mode == 1) inv /= 1.0f + expf(-__bfloat162float(gp[head]));
+    bf16* dst = out + (size_t)seq * out_stride + (size_t)head * D;
+#pragma unroll
+    for (int i = 0; i < (D + 31) / 32; ++i) {
+      const int d = lane + 32 * i;
+      if (d >= D) continue;
+      float v = acc[i] * inv;
+      if (gate_mode == 2) v /= 1.0f + expf(-__bfloat162float(gp[(size_t)head * D + d]));
+      dst[d] = __float2bfloat16_rn(v);
     }
   }
 }
@@ -865,7 +1027,6 @@ __host__ __device__ constexpr size_t fused_base_bytes(int stages) {
   return ((size_t)stages * 2 * TILE_ELEMS * sizeof(bf16) > (size_t)4 * 16 * (D + 2) * sizeof(float))
              ? (size_t)stages * 2 * TILE_ELEMS * sizeof(bf16) : (size_t)4 * 16 * (D + 2) * sizeof(float);
 }
-constexpr size_t PAGE_SMEM = (size_t)2 * 2 * TILE_ELEMS * sizeof(bf16);
 constexpr size_t RED_SMEM = (size_t)4 * 16 * (D + 2) * sizeof(float);
 constexpr size_t DECODE_SMEM = PAGE_SMEM > RED_SMEM ? PAGE_SMEM : RED_SMEM;
 
@@ -1681,6 +1842,46 @@ KRK_API int krk_sink_window_prefill(void* out, int out_stride, float out_scale, 
       (const bf16*)gate, gate_stride, gate_mode, slopes, softcap);
   KRK_CHECK_LAUNCH();
   return 0;
+}
+
+// The same for one token per sequence (row `seq` of the queries is sequence seq's), see sink_window_decode_kernel: `splits`
+// (up to 8) blocks of a cluster share an item's keys. -2: odd strides or offsets, or shared memory that does not fit.
+KRK_API int krk_sink_window_decode(void* out, int out_stride, float out_scale, const void* q_base, int q_stride, int HQ,
+                                   int HKV, const float* sink, const int* seq_slot, const int* seq_start, const int* table,
+                                   int width, const void* k_cache, const void* v_cache, int n_seqs, float scale, int window,
+                                   int keep_first, int keep_pages, const void* gate, int gate_stride, int gate_mode,
+                                   const float* slopes, float softcap, int splits, cudaStream_t stream) {
+  if (n_seqs == 0) return 0;
+  const int G = HQ / HKV, row_tiles = (G + 15) / 16, inbox_rows = G < 16 ? G : 16;
+  if ((q_stride & 1) || ((uintptr_t)q_base & 3) || splits < 1 || splits > 8) return -2;
+  if ((long long)HKV * row_tiles > 65535 || n_seqs > 65535) return -3;
+  const size_t smem = PAGE_SMEM + (size_t)splits * inbox_rows * (D + 2) * sizeof(float);
+  if (smem > 220 * 1024 || (size_t)4 * 16 * (D + 2) * sizeof(float) > PAGE_SMEM) return -2;
+  static size_t configured = 0;
+  if (smem > configured) {
+    cudaError_t e = cudaFuncSetAttribute(sink_window_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    configured = smem;
+  }
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(splits, HKV * row_tiles, n_seqs);
+  cfg.blockDim = dim3(THREADS);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = stream;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = splits;
+  attr[0].val.clusterDim.y = 1;
+  attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = 1;
+  static const bool plain = getenv("KRK_NO_PDL") != nullptr;
+  cfg.attrs = attr;
+  cfg.numAttrs = plain ? 1 : 2;
+  return (int)cudaLaunchKernelEx(&cfg, sink_window_decode_kernel, (bf16*)out, out_stride, out_scale, (const bf16*)q_base,
+                                 q_stride, HQ, HKV, sink, seq_slot, seq_start, table, width, (const bf16*)k_cache,
+                                 (const bf16*)v_cache, scale * LOG2E, window, keep_first, keep_pages, (const bf16*)gate,
+                                 gate_stride, gate_mode, slopes, softcap, row_tiles, inbox_rows);
 }
 
 // Attention with mixed head scores over blocks of keys, for steps of many tokens (see mixed_prefill_kernel). q_base,

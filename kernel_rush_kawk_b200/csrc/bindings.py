@@ -94,7 +94,7 @@ _MOE_SIGNATURES = {
     "krk_moe_down_pairs": [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, _P, c_int, _P, c_int, _P],
     "krk_moe_sort": [_P, _P, _P, c_int, c_int, c_int, _P],
     "krk_moe_gather": [_P, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, _P, _P, c_int, _P],
-    "krk_grouped_gemm": [_P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_float, c_float, _P, _P],
+    "krk_grouped_gemm": [_P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_float, c_float, _P, _P],
     "krk_moe_combine": [_P, _P, _P, _P, _P, _P, _P, c_int, _P, c_int, c_int, c_int, _P, c_int, _P, c_int, _P],
 }
 _MEMORY_SIGNATURES = {
@@ -132,6 +132,8 @@ _ATTN_SIGNATURES = {
                               c_int, _P],
     "krk_sink_window_prefill": [_P, c_int, c_float, _P, c_int, c_int, c_int, _P, _P, _P, _P, _P, _P, c_int, _P, _P, c_int,
                                 c_int, c_float, c_int, c_int, c_int, _P, c_int, c_int, _P, c_float, _P],
+    "krk_sink_window_decode": [_P, c_int, c_float, _P, c_int, c_int, c_int, _P, _P, _P, _P, c_int, _P, _P, c_int, c_float, c_int,
+                               c_int, c_int, _P, c_int, c_int, _P, c_float, c_int, _P],
     "krk_mixed_prefill": [_P, c_int, c_float, _P, c_int, c_int, c_int, _P, _P, _P, _P, _P, _P, _P, c_int, _P, _P, c_int,
                           c_int, c_float, c_int, _P, c_int, c_int, _P, c_int, _P],
     "krk_attention_decode": [_P, _P, c_int, c_int, c_int, _P, _P, _P, c_int, _P, _P, c_int, c_float, c_int, c_int, _P,
@@ -935,7 +937,7 @@ class Kernels:
     @staticmethod
     def _use_grouped(x, K, F, C, gated, activation) -> bool:
         """Whether the experts' products of many rows run as two grouped launches (sizes and alignment)."""
-        return ((not gated or activation == "swish_clamped") and x.dtype == torch.bfloat16 and K % 8 == 0 and F % 8 == 0 and C % 8 == 0 and min(K, F) >= 64)
+        return ((not gated or activation in ("swish_clamped", "silu")) and x.dtype == torch.bfloat16 and K % 8 == 0 and F % 8 == 0 and C % 8 == 0 and min(K, F) >= 64)
 
     def _grouped_experts(self, x, w_first, w_down, experts, w_in, w_out, activation, act_params, add, add_gate, gated, add_input,
                          offsets, place):
@@ -948,14 +950,17 @@ class Kernels:
         pairs = rows * top
         empty = lambda n: torch.empty((pairs, n), dtype=x.dtype, device=x.device)
         xg, h, yg = empty(K), empty(F), empty(C)
+        # blocks of up to 256 rows: experts of more than 128 rows on the average, and blocks enough for two rounds over the
+        # SMs all the same (4,096 rows of 16 experts of 512: 33 against 28 us; 12,288 of 64 of 1,408: 199 against 258 us)
+        tall = lambda n, cols: int(pairs > 128 * E and E * -(-n // cols) >= 296)
         row_w = torch.empty(pairs, dtype=torch.float32, device=x.device) if w_in is not None else None  # in the rows' new order
         self._ok(self.moe.krk_moe_gather(xg.data_ptr(), ptr, stride, place.data_ptr(), experts.data_ptr(), offsets.data_ptr(), 0,
                                          rows, top, K, _ptr(w_in), _ptr(row_w), _code(x.dtype), self._stream()), "expert gather")
         self._ok(self.moe.krk_grouped_gemm(h.data_ptr(), xg.data_ptr(), w_first.data_ptr(), offsets.data_ptr(), pairs, E, F, K,
-                                           _ACTIVATIONS[activation], int(gated), _ptr(row_w), float(act_params[0]),
+                                           _ACTIVATIONS[activation], int(gated), tall(F, 128 if gated else 256), _ptr(row_w), float(act_params[0]),
                                            float(act_params[1]), self.error.data_ptr(), self._stream()), "experts' first product")
         self._ok(self.moe.krk_grouped_gemm(yg.data_ptr(), h.data_ptr(), w_down.data_ptr(), offsets.data_ptr(), pairs, E, C, F, -1,
-                                           0, None, 0.0, 0.0, self.error.data_ptr(), self._stream()), "experts' second product")
+                                           0, tall(C, 256), None, 0.0, 0.0, self.error.data_ptr(), self._stream()), "experts' second product")
         out = torch.empty((rows, C), dtype=x.dtype, device=x.device)
         self._ok(self.moe.krk_moe_combine(out.data_ptr(), _ptr(add), _ptr(add_gate), yg.data_ptr(), place.data_ptr(),
                                           experts.data_ptr(), offsets.data_ptr(), 0, _ptr(w_out), rows, top, C, ptr, stride,
@@ -1026,12 +1031,31 @@ class Kernels:
             raise KernelError("the distance bias takes one float32 slope per query head")
         shape = (_ptr(slopes), float(softcap or 0.0))
         extras = (keep_first, keep_pages, g_ptr, g_stride, g_col, g_mode, *shape)
+        tensor_cores = (proj.dtype == torch.bfloat16 and dim == vdim == cache.v_dim and dim % 16 == 0 and dim <= 256
+                        and dim in self.attn)  # whole pages on the tensor cores, kernels compiled per head size
         if batch.is_decode and proj.shape[0] == batch.n_seqs:
             # one token per sequence: a block per (sequence, kv head), its warps splitting the window's keys. The
             # choice depends on the step's shape alone, so a sequence's results do not depend on its batch
             # blocks per (sequence, kv head) by the number of such items alone, never by lengths, so that a
             # captured step stays valid: enough to give every SM a block while items are few
             items = batch.n_seqs * cache.kv_heads
+            esz = proj.element_size()
+            if tensor_cores and not fuse and hasattr(self.attn[dim], "krk_sink_window_decode"):
+                # bfloat16, key and value heads of one size: whole pages on the tensor cores, an item's blocks a cluster
+                row_tiles = -(-(heads // cache.kv_heads) // 16)
+                tiles = items * row_tiles
+                pages = -(-min(int(window or 1 << 30), cache.width * 64) // 64) + 1 + -(-keep_first // 64)
+                splits = 8 if tiles <= 37 else 4 if tiles <= 74 else 2 if tiles <= 192 else 1
+                while splits > pages:
+                    splits //= 2
+                rc = self.attn[dim].krk_sink_window_decode(
+                    optr + out_col * esz, ostride, float(out_scale), ptr + q_col * esz, stride, heads, cache.kv_heads, _ptr(sink),
+                    batch.seq_slot.data_ptr(), batch.seq_start.data_ptr(), cache.table.data_ptr(), cache.width, cache.k.data_ptr(),
+                    cache.v.data_ptr(), batch.n_seqs, float(scale), int(window or 0), keep_first, keep_pages,
+                    None if g_ptr is None else g_ptr + g_col * esz, g_stride, g_mode, *shape, splits, self._stream())
+                if rc != -2:  # -2: odd strides or offsets, or too large for it; the kernel below takes them
+                    self._ok(rc, "tensor-core single-token windowed attention")
+                    return True
             splits = 8 if items <= 18 else 4 if items <= 37 else 2 if items <= 74 else 1
             key = ("sink", batch.n_seqs, heads, vdim, splits)
             scratch = self._partials.get(key)
@@ -1052,9 +1076,8 @@ class Kernels:
                 return False
         elif fuse:
             return False
-        if (proj.dtype == torch.bfloat16 and dim == vdim == cache.v_dim and dim % 16 == 0 and dim <= 256 and dim in self.attn
-                and not batch.is_decode and hasattr(self.attn[dim], "krk_sink_window_prefill")):
-            # many tokens per sequence in bfloat16: the tensor-core walk over whole pages (compiled per head size)
+        if tensor_cores and not batch.is_decode and hasattr(self.attn[dim], "krk_sink_window_prefill"):
+            # many tokens per sequence: the tensor-core walk over whole pages
             esz = proj.element_size()
             rc = self.attn[dim].krk_sink_window_prefill(
                 optr + out_col * esz, ostride, float(out_scale), ptr + q_col * esz, stride, heads, cache.kv_heads,

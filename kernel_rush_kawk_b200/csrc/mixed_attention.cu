@@ -77,6 +77,83 @@ __global__ void embed_bigram_kernel(float* __restrict__ out, const T* __restrict
   }
 }
 
+// what the queries at a position are multiplied by
+__device__ __forceinline__ float temperature(int pos, float coef, int every) {
+  return 1.0f + coef * logf((float)((pos + 1) / every + 1));
+}
+
+// four consecutive elements (or zeros)
+template <typename T> __device__ __forceinline__ void load4v(const T* p, float* f, bool on);
+template <> __device__ __forceinline__ void load4v<float>(const float* p, float* f, bool on) {
+  const float4 v = on ? *reinterpret_cast<const float4*>(p) : make_float4(0.f, 0.f, 0.f, 0.f);
+  f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+}
+template <> __device__ __forceinline__ void load4v<bf16>(const bf16* p, float* f, bool on) {
+  const uint2 raw = on ? *reinterpret_cast<const uint2*>(p) : make_uint2(0u, 0u);
+  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+  f[0] = __low2float(h[0]); f[1] = __high2float(h[0]); f[2] = __low2float(h[1]); f[3] = __high2float(h[1]);
+}
+template <typename T> __device__ __forceinline__ void store4v(T* p, const float* f);
+template <> __device__ __forceinline__ void store4v<float>(float* p, const float* f) {
+  *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+}
+template <> __device__ __forceinline__ void store4v<bf16>(bf16* p, const float* f) {
+  __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<unsigned*>(&a), *reinterpret_cast<unsigned*>(&b));
+}
+
+// What the kernel below does, for heads that are neither biased nor rotated, of a multiple of 4 elements up to 256: a lane keeps four
+// consecutive elements of every 128, one load and one store each.
+template <typename T>
+__global__ void norm_write_kernel(T* proj, int stride, int q_col, int k_col, int v_col, int HQ, int HKV, int D, int DV,
+                                  const float* __restrict__ gain, float eps, int unit, float temp_coef, int temp_every,
+                                  const int* __restrict__ row_seq, const int* __restrict__ row_pos,
+                                  const int* __restrict__ seq_slot, const int* __restrict__ table, int width, T* k_cache,
+                                  T* v_cache, int rows, int keep_pages) {
+  grid_launch_dependents();
+  const int lane = threadIdx.x & 31;
+  const int per_row = HQ + 2 * HKV;
+  const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (item >= (long long)rows * per_row) return;
+  const int row = (int)(item / per_row), which = (int)(item % per_row);
+  const bool query = which < HQ, key = !query && which < HQ + HKV;
+  const int h = query ? which : key ? which - HQ : which - HQ - HKV;
+  const int n = query || key ? D : DV;
+  const bool normed = (query || key) && (gain != nullptr || unit);
+  float g[2][4];
+#pragma unroll
+  for (int c = 0; c < 2; ++c) {  // weights, before the wait
+    const int e = 128 * c + 4 * lane;
+    if ((query || key) && gain && e < n) load4v<float>(gain + (key ? D : 0) + e, g[c], true);
+    else g[c][0] = g[c][1] = g[c][2] = g[c][3] = 1.f;
+  }
+  grid_dependency_wait();
+  const int pos = row_pos[row];
+  T* src = proj + (size_t)row * stride + (query ? q_col : key ? k_col : v_col) + (size_t)h * n;
+  float x[2][4];
+  float sq = 0.f;
+#pragma unroll
+  for (int c = 0; c < 2; ++c) {
+    load4v<T>(src + 128 * c + 4 * lane, x[c], 128 * c + 4 * lane < n);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) sq += x[c][i] * x[c][i];
+  }
+  T* dst = src;
+  if (!query) {
+    const int page = page_of(table, width, seq_slot[row_seq[row]], pos, keep_pages);
+    dst = (key ? k_cache : v_cache) + (((size_t)page * HKV + h) * KRK_PAGE + (pos % KRK_PAGE)) * n;
+  }
+  float f = normed ? rsqrtf(warp_sum(sq) / (float)n + eps) : 1.f;
+  if (query && temp_every > 0) f *= temperature(pos, temp_coef, temp_every);
+#pragma unroll
+  for (int c = 0; c < 2; ++c) {
+    if (128 * c + 4 * lane >= n) continue;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) x[c][i] = x[c][i] * f * g[c][i];
+    store4v<T>(dst + 128 * c + 4 * lane, x[c]);
+  }
+}
+
 template <typename T>
 __global__ void bias_norm_rotate_write_kernel(T* proj, int stride, int q_col, int k_col, int v_col, int HQ, int HKV, int D,
                                               int DV, const float* __restrict__ bias, const float* __restrict__ gain,
@@ -134,7 +211,7 @@ __global__ void bias_norm_rotate_write_kernel(T* proj, int stride, int q_col, in
     }
     rstd = rsqrtf(warp_sum(sq) / (float)n + eps);
   }
-  if (temp_every > 0 && which < HQ) rstd *= 1.0f + temp_coef * logf((float)((pos + 1) / temp_every + 1));
+  if (temp_every > 0 && which < HQ) rstd *= temperature(pos, temp_coef, temp_every);
   __syncwarp();  // q is rewritten in place: every lane has read what it needs of the head
   auto val = [&](int e) { return (to_float<T>(src[e]) + (b ? b[e] : 0.f)) * rstd * (g ? g[e] : 1.f); };
   const int half = turn >> 1;
@@ -180,18 +257,6 @@ template <> __device__ __forceinline__ float dot_key<bf16>(const float* q, const
     for (int d = 0; d < D; ++d) dot += q[d] * __bfloat162float(k[d]);
   }
   return dot;
-}
-
-// four consecutive elements of a value row (or zeros)
-template <typename T> __device__ __forceinline__ void load4v(const T* p, float* f, bool on);
-template <> __device__ __forceinline__ void load4v<float>(const float* p, float* f, bool on) {
-  const float4 v = on ? *reinterpret_cast<const float4*>(p) : make_float4(0.f, 0.f, 0.f, 0.f);
-  f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
-}
-template <> __device__ __forceinline__ void load4v<bf16>(const bf16* p, float* f, bool on) {
-  const uint2 raw = on ? *reinterpret_cast<const uint2*>(p) : make_uint2(0u, 0u);
-  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
-  f[0] = __low2float(h[0]); f[1] = __high2float(h[0]); f[2] = __low2float(h[1]); f[3] = __high2float(h[1]);
 }
 
 constexpr int MIX_VPL = 8;  // value heads up to 256
@@ -540,6 +605,17 @@ KRK_API int krk_bias_norm_rotate_write(void* proj, int stride, int q_col, int k_
   const int warps = 4;
   const long long blocks = (items + warps - 1) / warps;
   if (blocks > 0x7fffffffLL) return -3;
+  const size_t piece = dtype == KRK_DTYPE_F32 ? 16 : 8;
+  if (!bias && rot == 0 && D % 4 == 0 && DV % 4 == 0 && D <= 256 && DV <= 256 && stride % 4 == 0 && q_col % 4 == 0 &&
+      k_col % 4 == 0 && v_col % 4 == 0 && (uintptr_t)proj % piece == 0 && ((uintptr_t)gain & 15) == 0) {
+    if (dtype == KRK_DTYPE_F32)
+      return (int)launch_pdl(norm_write_kernel<float>, dim3((unsigned)blocks), dim3(warps * 32), 0, stream, (float*)proj,
+                             stride, q_col, k_col, v_col, HQ, HKV, D, DV, gain, eps, unit, temp_coef, temp_every, row_seq,
+                             row_pos, seq_slot, table, width, (float*)k_cache, (float*)v_cache, rows, keep_pages);
+    return (int)launch_pdl(norm_write_kernel<bf16>, dim3((unsigned)blocks), dim3(warps * 32), 0, stream, (bf16*)proj, stride,
+                           q_col, k_col, v_col, HQ, HKV, D, DV, gain, eps, unit, temp_coef, temp_every, row_seq, row_pos,
+                           seq_slot, table, width, (bf16*)k_cache, (bf16*)v_cache, rows, keep_pages);
+  }
   if (dtype == KRK_DTYPE_F32)
     return (int)launch_pdl(bias_norm_rotate_write_kernel<float>, dim3((unsigned)blocks), dim3(warps * 32), 0, stream,
                            (float*)proj, stride, q_col, k_col, v_col, HQ, HKV, D, DV, bias, gain, eps, unit, temp_coef, temp_every, inv_freq, rot, pairs,

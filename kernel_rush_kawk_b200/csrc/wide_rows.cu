@@ -21,24 +21,6 @@
 
 namespace {
 
-template <typename T>
-__global__ void embed_scaled_kernel(float* __restrict__ out, const T* __restrict__ table, const int* __restrict__ ids,
-                                    int H, int n_table_rows, float scale, int* error, int copies, T* __restrict__ rounded) {
-  grid_launch_dependents();
-  grid_dependency_wait();
-  const int r = blockIdx.x;
-  const int id = ids[r];
-  const bool bad = id < 0 || id >= n_table_rows;
-  if (bad && threadIdx.x == 0 && error) atomicExch(error, 1);
-  const T* src = table + (size_t)(bad ? 0 : id) * H;
-  float* dst = out + (size_t)r * H * copies;  // the row is written `copies` times side by side
-  for (int i = threadIdx.x; i < H; i += blockDim.x) {
-    const float v = bad ? 0.f : to_float<T>(src[i]) * scale;
-    for (int c = 0; c < copies; ++c) dst[(size_t)c * H + i] = v;
-    if (rounded) rounded[(size_t)r * H + i] = from_float<T>(v);  // the same row as the first sublayer reads it
-  }
-}
-
 template <typename T> __device__ __forceinline__ void load4_rows(const T* p, float* f);
 template <> __device__ __forceinline__ void load4_rows<float>(const float* p, float* f) {
   const float4 v = *reinterpret_cast<const float4*>(p);
@@ -59,6 +41,36 @@ template <> __device__ __forceinline__ void store4_rows<bf16>(bf16* p, const flo
   raw.x = *reinterpret_cast<unsigned*>(&a);
   raw.y = *reinterpret_cast<unsigned*>(&b);
   *reinterpret_cast<uint2*>(p) = raw;
+}
+
+template <typename T>
+__global__ void embed_scaled_kernel(float* __restrict__ out, const T* __restrict__ table, const int* __restrict__ ids,
+                                    int H, int n_table_rows, float scale, int* error, int copies, T* __restrict__ rounded) {
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int r = blockIdx.x;
+  const int id = ids[r];
+  const bool bad = id < 0 || id >= n_table_rows;
+  if (bad && threadIdx.x == 0 && error) atomicExch(error, 1);
+  const T* src = table + (size_t)(bad ? 0 : id) * H;
+  float* dst = out + (size_t)r * H * copies;  // the row is written `copies` times side by side
+  if (copies == 1 && (H & 3) == 0) {  // rows of the table and of the results then start on 8- or 16-byte boundaries
+    for (int i = 4 * (blockIdx.y * blockDim.x + threadIdx.x); i < H; i += 4 * gridDim.y * blockDim.x) {
+      float v[4] = {0.f, 0.f, 0.f, 0.f};
+      if (!bad) load4_rows<T>(src + i, v);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) v[j] *= scale;
+      store4_rows<float>(dst + i, v);
+      if (rounded) store4_rows<T>(rounded + (size_t)r * H + i, v);
+    }
+    return;
+  }
+  if (blockIdx.y > 0) return;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    const float v = bad ? 0.f : to_float<T>(src[i]) * scale;
+    for (int c = 0; c < copies; ++c) dst[(size_t)c * H + i] = v;
+    if (rounded) rounded[(size_t)r * H + i] = from_float<T>(v);  // the same row as the first sublayer reads it
+  }
 }
 
 template <typename T, bool VEC>
@@ -292,14 +304,18 @@ __global__ void gated_act_kernel(T* __restrict__ out, const T* __restrict__ gu, 
 
 }  // namespace
 
+static dim3 embed_grid(int rows, int H, int copies) {  // a piece of four elements a thread where a row is cut that way
+  return dim3(rows, copies == 1 && (H & 3) == 0 ? (H / 4 + 127) / 128 : 1);
+}
+
 KRK_API int krk_embed_scaled(float* out, const void* table, const int* ids, int rows, int H, int n_table_rows, float scale,
                              int* error, int dtype, cudaStream_t stream, int copies, void* rounded) {
   if (rows == 0) return 0;
   if (copies < 1) return -2;
   if (dtype == KRK_DTYPE_F32)
-    return (int)launch_pdl(embed_scaled_kernel<float>, dim3(rows), dim3(128), 0, stream, out, (const float*)table, ids, H,
+    return (int)launch_pdl(embed_scaled_kernel<float>, embed_grid(rows, H, copies), dim3(128), 0, stream, out, (const float*)table, ids, H,
                            n_table_rows, scale, error, copies, (float*)rounded);
-  return (int)launch_pdl(embed_scaled_kernel<bf16>, dim3(rows), dim3(128), 0, stream, out, (const bf16*)table, ids, H,
+  return (int)launch_pdl(embed_scaled_kernel<bf16>, embed_grid(rows, H, copies), dim3(128), 0, stream, out, (const bf16*)table, ids, H,
                          n_table_rows, scale, error, copies, (bf16*)rounded);
 }
 

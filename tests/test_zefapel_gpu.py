@@ -454,7 +454,7 @@ def test_grouped_products_where_experts_have_few_rows_many_or_none():
             out = torch.full((rows + 5, N), 7.0, dtype=torch.bfloat16, device="cuda")
             a_d, w_d, o_d = a.cuda(), w.cuda(), offsets.cuda()
             rt.ops._ok(rt.ops.moe.krk_grouped_gemm(out.data_ptr(), a_d.data_ptr(), w_d.data_ptr(), o_d.data_ptr(), rows + 5, E, N, K,
-                                                   act, rt.ops.error.data_ptr(), rt.ops._stream()), "grouped product")
+                                                   act, 0, 0, None, 0.0, 0.0, rt.ops.error.data_ptr(), rt.ops._stream()), "grouped product")
             want = torch.full((rows + 5, N), 7.0, dtype=torch.float64)
             for e in range(E):
                 lo, hi = int(offsets[e]), int(offsets[e + 1])
