@@ -9,8 +9,8 @@
 // The tile engine is that of gemm_tcgen05.cu: warp 0 drives TMA (128 rows of A, BN rows of W, 64 elements of K a stage,
 // 128-byte swizzle), warp 1 owns tensor memory and issues tcgen05.mma, warps 2..5 read the accumulator back. With MT = 2 a
 // block takes up to 256 of an expert's rows: two tiles of A ride with every tile of W into two accumulators (all 512 columns
-// of tensor memory), which warps 2..5 and 6..9 read back side by side; what bounds the kernel where experts have more than
-// one tile of rows is the operands' way out of the L2 cache, and W then makes it once instead of twice. A tile of A
+// of tensor memory), which warps 2..5 and 6..9 read back side by side. Where experts have more than one tile of rows, W is
+// then fetched once instead of twice and half as many blocks pay for their start and their epilogue. A tile of A
 // that reaches past its expert's rows reads the next expert's (or zeros beyond the matrix); what it makes of them is not
 // stored. Every wait is bounded: one that runs out sets the error word and the block leaves, after freeing its tensor
 // memory.
